@@ -22,7 +22,7 @@
 extern "C" {
 #endif
 
-#define LL_ABI_VERSION 15
+#define LL_ABI_VERSION 16
 
 #define LL_OK 0
 #define LL_ERR_ARG (-1)         /* bad shape / dtype / null pointer */
@@ -371,6 +371,10 @@ LL_API int ll_gain_norm_add_mix(const float* x, const void* y, int y_dtype, cons
  *   g = min(gu[c], limit), u = clamp(gu[ff + c], -limit, limit), h[c] = g * sigmoid(alpha * g) * (u + 1). */
 LL_API int ll_glu_clamp(const void* gu, int gu_stride, int ff, float limit, float alpha, void* h, int dtype, int rows,
                         ll_stream stream);
+/* The same with the shift of the up branch as a parameter: h[c] = g * sigmoid(alpha * g) * (u + shift)  (limit +inf, alpha 1,
+ * shift 0: the plain silu-gated unit). */
+LL_API int ll_glu_unit(const void* gu, int gu_stride, int ff, float limit, float alpha, float shift, void* h, int dtype, int rows,
+                       ll_stream stream);
 
 /* ---------------------------------------------------------------------------------------
  * Latent attention over a ring cache of latent rows (csrc/latent_attn.cu).  A cache row is
@@ -417,17 +421,27 @@ LL_API int ll_moe_route_scored(const void* x, int dtype, const float* w_router, 
                                int top, int score_all, int n_groups, int keep_groups, int32_t* expert_idx, float* expert_w,
                                int32_t* counts, int32_t* rank, int32_t* offsets, int32_t* perm, ll_stream stream);
 
+/* The same with every rule of the choice as a parameter.  score 0 / 1: as score_all above.  score 2: scores = sigmoid(z), the
+ * experts compete by score + correction[e] (fp32 [X], NULL: none), expert_w = chosen scores without the correction / (their sum
+ * + 1e-20).  In every case expert_w is multiplied by out_scale.  group_top: a group's score is its largest choice score (1) or
+ * the sum of its two largest (2). */
+LL_API int ll_moe_route_choice(const void* x, int dtype, const float* w_router, const float* bias, int M, int dim, int n_experts,
+                               int top, int score, const float* correction, float out_scale, int n_groups, int keep_groups,
+                               int group_top, int32_t* expert_idx, float* expert_w, int32_t* counts, int32_t* rank,
+                               int32_t* offsets, int32_t* perm, ll_stream stream);
+
 /* Grouped GEMM over the sorted rows, one expert's weight per row segment; w is the experts' stack.
  * mode 1: w [X][2N][K] = [gate; up]; a [M][lda] read at token perm[r] / top;
  *         c[r][:] = glu(a . gate^T, a . up^T) with ll_glu_clamp's formula, rows in sorted order.
  * mode 2: as mode 1 with the up branch entering as it is: g * sigmoid(alpha g) * u (limit +inf: no clamp; alpha 1: silu).
+ * mode 3: w [X][N][K]; a read as in mode 1; c[r][:] = relu(a . w[e]^T)^2, rows in sorted order.
  * mode 0: w [X][N][K]; a [n_rows][lda] in sorted order; c[perm[r]][:] = a[r] . w[e]^T. */
 LL_API int ll_moe_grouped_gemm(const void* a, int lda, const void* w, const int32_t* offsets, const int32_t* perm, int mode,
                                int dtype, int n_rows, int top, int n_experts, int N, int K, float limit, float alpha,
                                void* c, int ldc, ll_stream stream);
 
 /* The same grouped GEMM on the tcgen05 tensor cores (bf16, TMA-tiled operands, accumulators in TMEM), for steps with
- * many rows per expert.  a [n_rows][K] holds the rows ALREADY in sorted order (mode 1: gather them with
+ * many rows per expert.  a [n_rows][K] holds the rows ALREADY in sorted order (modes 1 to 3: gather them with
  * ll_moe_gather_rows: out[r] = x[perm[r] / top]); w, offsets, perm, mode, c as in ll_moe_grouped_gemm.  K a multiple of 8,
  * operands 16-byte aligned.  ll_moe_tc_error(): 0, or the code of the first bounded wait that ran out inside these
  * kernels since the library was loaded (synchronises the device). */
@@ -450,6 +464,10 @@ LL_API int ll_moe_combine(const void* y, const float* expert_w, int top, const v
 LL_API int ll_add_norm_pair(float* x, const void* a0, float s0, const void* a1, float s1, const void* a2, float s2, const float* w1,
                             const float* w2, float eps, void* out1, int out1_f32, void* out2, int act_dtype, int rows, int dim,
                             ll_stream stream);
+/* x[m][:] += s * a (optional, activation dtype), in place, fp32; then, with out given, the layer norm of the same row:
+ * out = (x - mean) / sqrt(var + eps) * w + b, var the mean squared deviation (w, b fp32 [dim]; out in the activation dtype). */
+LL_API int ll_add_layer_norm(float* x, const void* a, float s, const float* w, const float* b, float eps, void* out, int act_dtype,
+                             int rows, int dim, ll_stream stream);
 /* RMS norm of fp32 rows y in `groups` equal parts with a gate (activation dtype, row stride gate_stride; silu, or a sigmoid
  * when gate_sigmoid):  gate_first 1: (y * gate(g)) / rms_part(.) * w;  0: y / rms_part(y) * w * gate(g).  w: C entries, or
  * C / groups shared by the parts (w_shared).  A part of y spans y_gs numbers (0: C / groups), of which the first C / groups are
@@ -505,6 +523,11 @@ LL_API int ll_decay_scan(const void* q, int q_stride, const void* k, int k_strid
                          const float* a, int a_per_channel, const float* ks, const float* skip, float qs, float* state,
                          const int32_t* pos_ids, float* y, int B, int T, int H, int qk_heads, int n, int p, int unit_col,
                          ll_stream stream);
+/* The same walk with one constant decay per head (a fp32 [H]), no key scale and no skip; act_silu: q, k and v pass silu as they
+ * are read (rounded to the activation dtype). */
+LL_API int ll_decay_scan_constant(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, int dtype,
+                                  const float* a, int act_silu, float qs, float* state, const int32_t* pos_ids, float* y, int B, int T,
+                                  int H, int qk_heads, int n, int p, ll_stream stream);
 /* Exponential gates with a running stabiliser, per (b, h): li = cap(raw_i + bias_i[h]), lf = logsigmoid(cap(raw_f + bias_f[h])),
  * cap(z) = c tanh(z / c) (c <= 0: none); mx_t = max(lf_t + mx_(t-1), li_t) with mx carried in mstate fp32 [B][H] (0 when
  * pos_ids[0] == 0); keep = exp(lf + mx_(t-1) - mx_t), take = exp(li - mx_t), stab = mx_t   (fp32 [B*T][H] each). */
@@ -566,11 +589,26 @@ LL_API int ll_qk_rotary_append_maps(const void* q, int q_stride, const void* k, 
                                     const float* q_norm, const float* k_norm, float eps, const float* freq, int rot_dims,
                                     const int32_t* pos_ids, void* q_out, void* kc, void* vc, int B, int T, int H, int G, int dim,
                                     int vdim, int ring, int maps, ll_stream stream);
+/* Rows of this step with a norm per head: every head of q and k is divided by its own root mean square and multiplied by q_norm /
+ * k_norm (fp32 [dim], shared by the heads; NULL: no norm), the queries are multiplied by 1 + temp_coef * ln(floor((p + 1) /
+ * temp_every) + 1) at position p (temp_every 0: not), then the first rot_dims dimensions turn as in ll_qk_rotary_append.  The value
+ * row is v, or (1 - lam) * v + lam * first when `first` (another layer's values of the same tokens, [B*T][first_stride]) is given. */
+LL_API int ll_qk_head_append(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const void* first,
+                             int first_stride, float lam, int dtype, const float* q_norm, const float* k_norm, float eps,
+                             const float* freq, int rot_dims, float temp_coef, int temp_every, const int32_t* pos_ids, void* q_out,
+                             void* kc, void* vc, int B, int T, int H, int G, int dim, int vdim, int ring, ll_stream stream);
 LL_API int ll_softmax_attn_tensor_form(int dtype, int T, int dim, int vdim, int q_stride, int gate_stride, int splits);
 LL_API int ll_softmax_attn_maps(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, int dtype,
                                 const int32_t* pos_ids, const float* sink, float scale, float softcap, int B, int T, int H, int G,
                                 int dim, int vdim, int window, int chunk, int ring, int splits, int form, int maps, float diff_lambda,
                                 float diff_post, float eps, float* scratch, void* y, ll_stream stream);
+/* The same with a bias linear in the distance: s_h(i,j) = scale q_h(i).k_g(j) - slopes[h] * (i - j) (fp32 [H], shared by a head's
+ * maps; NULL: none) before the cap.  Slopes with maps > 1 take the fp32 form (scratch). */
+LL_API int ll_softmax_attn_biased(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc,
+                                  int dtype, const int32_t* pos_ids, const float* sink, const float* slopes, float scale,
+                                  float softcap, int B, int T, int H, int G, int dim, int vdim, int window, int chunk, int ring,
+                                  int splits, int form, int maps, float diff_lambda, float diff_post, float eps, float* scratch,
+                                  void* y, ll_stream stream);
 
 #ifdef __cplusplus
 }

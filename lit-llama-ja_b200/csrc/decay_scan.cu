@@ -12,6 +12,9 @@
 // unit_col: the LAST of the p columns of every head is not in memory but the constant 1 (v then holds p - 1 columns per
 // head).  That column of S is the running sum of the keys alone and that column of y its product with the query: the
 // normaliser of a matrix memory, carried by the same walk.
+//
+// A decay that is one constant per head (a_t = a[h] for every token) is read with a row stride of 0.  SILU: q, k and v are
+// silu'd as they are staged, rounded to the activation dtype as a kernel of its own would leave them.
 #include "common.cuh"
 
 namespace llb {
@@ -24,11 +27,18 @@ __host__ __device__ constexpr int ds_tc(int npad) { return npad <= 64 ? 16 : npa
 // columns per block.  A thread's rows are interleaved in quads, row(k, e) = (k * NP + part) * 4 + e, so that the NP lanes of
 // a column read consecutive 16-byte units of the staged token (no bank conflicts).
 // DS_NL: state rows a thread keeps in registers (8: more threads per head, the usual case; 16: heads of more than 256 rows).
-// PERCH: a decay per state row (gated linear attention); otherwise one per head and token, read once per token.
-template <typename T, int NP, int DS_NL, bool PERCH>
+// PERCH: a decay per state row (gated linear attention); otherwise one per head and token, read once per token (a_row: numbers
+// between two tokens' decays; 0: the same decays for every token).
+template <typename T, bool SILU>
+__device__ __forceinline__ float ds_in(T raw) {
+  const float x = dt<T>::ld(&raw, 0);
+  return SILU ? dt<T>::rd(x / (1.f + expf(-x))) : x;
+}
+
+template <typename T, int NP, int DS_NL, bool PERCH, bool SILU>
 __global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(
     const T* __restrict__ q, int q_stride, const T* __restrict__ k, int k_stride, const T* __restrict__ v, int v_stride,
-    const float* __restrict__ a, int a_per_channel, const float* __restrict__ ks, const float* __restrict__ skip, float qs,
+    const float* __restrict__ a, int a_row, const float* __restrict__ ks, const float* __restrict__ skip, float qs,
     float* __restrict__ state, const int32_t* __restrict__ pos_ids, float* __restrict__ y, int Tn, int H, int qk_heads, int n,
     int p, int vw) {
   constexpr int PT = DS_THREADS / NP;
@@ -60,7 +70,7 @@ __global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(
       const int tt = idx / NPAD, i = idx - tt * NPAD;
       const size_t m = (size_t)b * Tn + t0 + tt;
       const bool ok = t0 + tt < Tn && i < n;
-      ra[it] = ok ? (a_per_channel ? a[(m * H + h) * n + i] : a[m * H + h]) : 1.f;
+      ra[it] = ok ? (PERCH ? a[(m * H + h) * n + i] : a[m * a_row + h]) : 1.f;
       rs[it] = (ok && ks) ? ks[m * H + h] : 1.f;
       rk[it] = k[ok ? m * k_stride + (size_t)g * n + i : 0];
       rq[it] = q[ok ? m * q_stride + (size_t)g * n + i : 0];
@@ -84,8 +94,8 @@ __global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(
       const int tt = idx / NPAD, i = idx - tt * NPAD;
       const bool ok = t0 + tt < Tn && i < n;
       s_a[tt][i] = ra[it];
-      s_k[tt][i] = ok ? dt<T>::ld(&rk[it], 0) * rs[it] : 0.f;
-      s_q[tt][i] = ok ? dt<T>::ld(&rq[it], 0) * qs : 0.f;
+      s_k[tt][i] = ok ? ds_in<T, SILU>(rk[it]) * rs[it] : 0.f;
+      s_q[tt][i] = ok ? ds_in<T, SILU>(rq[it]) * qs : 0.f;
     }
 #pragma unroll
     for (int it = 0; it < VIT; ++it) {
@@ -93,7 +103,7 @@ __global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(
       const int tt = idx / PT, cc = idx - tt * PT;
       if (tt < DS_TC) {
         const int col = blockIdx.x * PT + cc;
-        s_v[tt][cc] = (t0 + tt < Tn && col < p) ? (col < vw ? dt<T>::ld(&rv[it], 0) : 1.f) : 0.f;
+        s_v[tt][cc] = (t0 + tt < Tn && col < p) ? (col < vw ? ds_in<T, SILU>(rv[it]) : 1.f) : 0.f;
       }
     }
     __syncthreads();
@@ -101,7 +111,6 @@ __global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(
     for (int tt = 0; tt < nt; ++tt) {
       const float vv = s_v[tt][pl];
       float c0 = 0.f, c1 = 0.f, c2 = 0.f, c3 = 0.f;
-#pragma unroll
       const float a1 = s_a[tt][0];
 #pragma unroll
       for (int i4 = 0; i4 < DS_NL; i4 += 4) {
@@ -132,18 +141,24 @@ __global__ void __launch_bounds__(DS_THREADS) decay_scan_kernel(
 #undef DS_ROW
 }
 
+// what the decays are: one per head and token, one per head, token and state row, or one constant per head
+enum DecayKind { DECAY_TOKEN, DECAY_CHANNEL, DECAY_HEAD };
+
 template <typename T, int NP, int NL>
 static int decay_scan_launch(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const float* a,
-                             int a_per_channel, const float* ks, const float* skip, float qs, float* state, const int32_t* pos_ids,
-                             float* y, int B, int Tn, int H, int qk_heads, int n, int p, int vw, cudaStream_t st) {
+                             DecayKind kind, bool silu, const float* ks, const float* skip, float qs, float* state,
+                             const int32_t* pos_ids, float* y, int B, int Tn, int H, int qk_heads, int n, int p, int vw, cudaStream_t st) {
   constexpr int PT = DS_THREADS / NP;
   const dim3 grid((p + PT - 1) / PT, H, B);
-  if (a_per_channel)
-    decay_scan_kernel<T, NP, NL, true><<<grid, DS_THREADS, 0, st>>>((const T*)q, q_stride, (const T*)k, k_stride, (const T*)v, v_stride, a, 1,
-                                                                    ks, skip, qs, state, pos_ids, y, Tn, H, qk_heads, n, p, vw);
-  else
-    decay_scan_kernel<T, NP, NL, false><<<grid, DS_THREADS, 0, st>>>((const T*)q, q_stride, (const T*)k, k_stride, (const T*)v, v_stride, a, 0,
-                                                                     ks, skip, qs, state, pos_ids, y, Tn, H, qk_heads, n, p, vw);
+  const int a_row = kind == DECAY_HEAD ? 0 : H;
+#define LL_DSK(PERCH, SILU)                                                                                                            \
+  decay_scan_kernel<T, NP, NL, PERCH, SILU><<<grid, DS_THREADS, 0, st>>>((const T*)q, q_stride, (const T*)k, k_stride, (const T*)v,    \
+                                                                         v_stride, a, a_row, ks, skip, qs, state, pos_ids, y, Tn, H,   \
+                                                                         qk_heads, n, p, vw)
+  if (kind == DECAY_CHANNEL) LL_DSK(true, false);
+  else if (silu) LL_DSK(false, true);
+  else LL_DSK(false, false);
+#undef LL_DSK
   LL_LAUNCH_OK("decay_scan_kernel");
   return LL_OK;
 }
@@ -250,15 +265,10 @@ __global__ void __launch_bounds__(MG_THREADS) matrix_memory_gates_kernel(
   if (threadIdx.x == 0) mstate[w] = mx;
 }
 
-}  // namespace llb
-
-using namespace llb;
-
-extern "C" {
-
-int ll_decay_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, int dtype, const float* a,
-                  int a_per_channel, const float* ks, const float* skip, float qs, float* state, const int32_t* pos_ids, float* y,
-                  int B, int T, int H, int qk_heads, int n, int p, int unit_col, ll_stream stream) {
+static int decay_scan_dispatch(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, int dtype,
+                               const float* a, DecayKind kind, bool silu, const float* ks, const float* skip, float qs, float* state,
+                               const int32_t* pos_ids, float* y, int B, int T, int H, int qk_heads, int n, int p, int unit_col,
+                               cudaStream_t st) {
   LL_CHECK_ARG(q && k && v && a && state && pos_ids && y, "decay_scan: null pointer");
   LL_CHECK_ARG(B >= 0 && T >= 0 && H > 0 && qk_heads > 0 && H % qk_heads == 0 && n > 0 && p > (unit_col ? 1 : 0),
                "bad decay_scan arguments");
@@ -268,7 +278,6 @@ int ll_decay_scan(const void* q, int q_stride, const void* k, int k_stride, cons
     return LL_ERR_UNSUPPORTED;
   }
   if (B == 0 || T == 0) return LL_OK;
-  cudaStream_t st = (cudaStream_t)stream;
   // 16 rows per thread when that already gives half of the SMs a block (each block stages its head's tokens: fewer blocks,
   // less staging); 8 rows when the heads are few, so that twice as many warps share the latency of the sequential walk
   int np16 = 1;
@@ -278,9 +287,9 @@ int ll_decay_scan(const void* q, int q_stride, const void* k, int k_stride, cons
   int np = 1;
   while (np * nl < n) np *= 2;
 #define LL_DS(TT, NP)                                                                                                                 \
-  return nl == 8 ? decay_scan_launch<TT, NP, 8>(q, q_stride, k, k_stride, v, v_stride, a, a_per_channel, ks, skip, qs, state, pos_ids, \
+  return nl == 8 ? decay_scan_launch<TT, NP, 8>(q, q_stride, k, k_stride, v, v_stride, a, kind, silu, ks, skip, qs, state, pos_ids, \
                                                 y, B, T, H, qk_heads, n, p, vw, st)                                                        \
-                 : decay_scan_launch<TT, NP, 16>(q, q_stride, k, k_stride, v, v_stride, a, a_per_channel, ks, skip, qs, state, pos_ids, \
+                 : decay_scan_launch<TT, NP, 16>(q, q_stride, k, k_stride, v, v_stride, a, kind, silu, ks, skip, qs, state, pos_ids, \
                                                  y, B, T, H, qk_heads, n, p, vw, st)
 #define LL_DS_T(TT)                 \
   switch (np) {                     \
@@ -297,6 +306,26 @@ int ll_decay_scan(const void* q, int q_stride, const void* k, int k_stride, cons
 #undef LL_DS
   set_error("decay_scan: unsupported dtype %d", dtype);
   return LL_ERR_UNSUPPORTED;
+}
+
+}  // namespace llb
+
+using namespace llb;
+
+extern "C" {
+
+int ll_decay_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, int dtype, const float* a,
+                  int a_per_channel, const float* ks, const float* skip, float qs, float* state, const int32_t* pos_ids, float* y,
+                  int B, int T, int H, int qk_heads, int n, int p, int unit_col, ll_stream stream) {
+  return decay_scan_dispatch(q, q_stride, k, k_stride, v, v_stride, dtype, a, a_per_channel ? DECAY_CHANNEL : DECAY_TOKEN, false, ks, skip,
+                             qs, state, pos_ids, y, B, T, H, qk_heads, n, p, unit_col, (cudaStream_t)stream);
+}
+
+int ll_decay_scan_constant(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, int dtype,
+                           const float* a, int act_silu, float qs, float* state, const int32_t* pos_ids, float* y, int B, int T, int H,
+                           int qk_heads, int n, int p, ll_stream stream) {
+  return decay_scan_dispatch(q, q_stride, k, k_stride, v, v_stride, dtype, a, DECAY_HEAD, act_silu != 0, nullptr, nullptr, qs, state, pos_ids,
+                             y, B, T, H, qk_heads, n, p, 0, (cudaStream_t)stream);
 }
 
 int ll_ssm_gates(const void* raw, int dtype, int stride, const float* dt_bias, const float* a_log, float* dt_out, float* decay,

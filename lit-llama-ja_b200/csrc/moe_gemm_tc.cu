@@ -5,11 +5,13 @@
 // gathered into that order once (ll_moe_gather_rows), so every operand is a plain row-major matrix
 // that TMA can tile:
 //   mode 1 (GLU) : h[r][n] = glu(xs[r] . gate_e[n], xs[r] . up_e[n])     w [X][2N][K] = [gate; up]
+//   mode 3 (relu^2): h[r][n] = relu(xs[r] . up_e[n])^2                    w [X][N][K]
 //   mode 0 (down): y[perm[r]][n] = h[r] . down_e[n]                       w [X][N][K]
 // for the sorted rows r of expert e.  A CTA owns 128 sorted rows of ONE expert (found from the device-side
 // offsets, as in the mma.sync form: no host synchronisation) x 256 accumulator columns in TMEM:
 //   GLU : columns 0..127 = gate tile, 128..255 = up tile of the same 128 outputs; the clamped gated unit is
 //         the epilogue, applied to the two accumulators as they are read back from TMEM;
+//   relu^2: columns 0..255 = 256 outputs, squared as they are read back;
 //   down: columns 0..255 = 256 outputs, scattered to (token, choice) order by the epilogue.
 // A row tile may run past its expert's last row: those rows (the next expert's, or zero fill) are
 // computed and never stored.
@@ -137,7 +139,7 @@ __global__ void __launch_bounds__(192, 2) moe_gemm_tc_kernel(const __grid_consta
     if (waited && *s_fail == 0) {
       const bool row_ok = rt < cnt;
       long long dst_row = 0;
-      if (row_ok) dst_row = MODE == 1 ? (long long)(r0 + rt) : (long long)perm[r0 + rt];
+      if (row_ok) dst_row = MODE != 0 ? (long long)(r0 + rt) : (long long)perm[r0 + rt];
       __nv_bfloat16* dst = c + dst_row * ldc;
       const uint32_t trow = tmem_d + ((uint32_t)(quarter * 32) << 16);
       constexpr int NCOL = MODE == 1 ? MT_BN : 2 * MT_BN;
@@ -158,7 +160,10 @@ __global__ void __launch_bounds__(192, 2) moe_gemm_tc_kernel(const __grid_consta
           }
         } else {
 #pragma unroll
-          for (int j = 0; j < 32; ++j) f[j] = __uint_as_float(v[j]);
+          for (int j = 0; j < 32; ++j) {
+            f[j] = __uint_as_float(v[j]);
+            if (MODE == 3) f[j] = fmaxf(f[j], 0.f) * fmaxf(f[j], 0.f);
+          }
         }
         if (!row_ok) continue;
         const int col = n0 + c0;
@@ -231,7 +236,7 @@ int ll_moe_gather_rows(const void* x, int ldx, const int32_t* perm, int top, int
 int ll_moe_grouped_gemm_tc(const void* a, const void* w, const int32_t* offsets, const int32_t* perm, int mode, int n_rows,
                            int n_experts, int N, int K, float limit, float alpha, void* c, int ldc, ll_stream stream) {
   LL_CHECK_ARG(a && w && offsets && perm && c, "moe_grouped_gemm_tc: null pointer");
-  LL_CHECK_ARG(n_rows >= 0 && n_experts > 0 && N > 0 && K > 0 && ldc >= N && mode >= 0 && mode <= 2, "bad moe_grouped_gemm_tc arguments");
+  LL_CHECK_ARG(n_rows >= 0 && n_experts > 0 && N > 0 && K > 0 && ldc >= N && mode >= 0 && mode <= 3, "bad moe_grouped_gemm_tc arguments");
   const float shift = mode == 2 ? 0.f : 1.f;     // mode 2: the up branch enters as it is
   if (mode == 2) mode = 1;
   LL_CHECK_ARG(K % 8 == 0 && ((uintptr_t)a & 15) == 0 && ((uintptr_t)w & 15) == 0 && ((uintptr_t)c & 15) == 0,
@@ -244,6 +249,7 @@ int ll_moe_grouped_gemm_tc(const void* a, const void* w, const int32_t* offsets,
   if (int r = make_map(w, (int)wrows, K, MT_BN, &mb)) return r;
   cudaStream_t st = (cudaStream_t)stream;
   if (mode == 1) return launch_moe_tc<1>(ma, mb, offsets, perm, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st);
+  if (mode == 3) return launch_moe_tc<3>(ma, mb, offsets, perm, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st);
   return launch_moe_tc<0>(ma, mb, offsets, perm, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st);
 }
 

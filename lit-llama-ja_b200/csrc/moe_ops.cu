@@ -5,9 +5,12 @@
 //
 //   route    z = W_r x + b (fp32), the `top` largest logits, weights = softmax over the chosen logits; or scores =
 //            softmax over ALL experts with weights = chosen scores / (their sum + 1e-20); optionally only experts of the
-//            `keep_groups` best of `n_groups` equal groups of neighbouring experts (a group's score: its largest) compete
+//            `keep_groups` best of `n_groups` equal groups of neighbouring experts (a group's score: its largest) compete;
+//            or scores = sigmoid(z), the choice made by score + correction (a group's score: the sum of its two largest
+//            choice scores), weights = chosen scores without the correction / (their sum + 1e-20) * a constant
 //   permute  rows sorted by expert: perm[offsets[e] + rank] = token * top + choice
 //   grouped  MODE_GLU : h[r][:] = glu(x[token(r)] . Wgu[e]^T)   (stacked [gate; up] weight; g s(alpha g) (u + shift), clamped)
+//            MODE_RELU2: h[r][:] = relu(x[token(r)] . Wu[e]^T)^2
 //            MODE_DOWN: y[perm[r]][:] = h[r] . Wd[e]^T
 //   combine  out[m] = sum_k w[m][k] * y[m * top + k]  (+ sigmoid(s[m]) * shared[m])
 #include "common.cuh"
@@ -17,17 +20,20 @@ namespace llb {
 constexpr int RT_TOK = 4;        // tokens per routing block
 constexpr int RT_THREADS = 256;
 constexpr int RT_EG = 4;         // experts a warp accumulates side by side
+enum { SCORE_CHOSEN = 0, SCORE_ALL = 1, SCORE_SIGMOID = 2 };
 
 template <typename T>
 __global__ void __launch_bounds__(RT_THREADS) moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w_router,
                                                                const float* __restrict__ bias, int M, int dim, int X, int top,
-                                                               int score_all, int n_groups, int keep_groups,
+                                                               int score, const float* __restrict__ correction, float out_scale,
+                                                               int n_groups, int keep_groups, int group_top,
                                                                int32_t* __restrict__ expert_idx, float* __restrict__ expert_w,
                                                                int32_t* __restrict__ counts, int32_t* __restrict__ rank) {
   extern __shared__ float sm[];
   float* xs = sm;                      // [RT_TOK][dim]
   float* zs = xs + RT_TOK * dim;       // [RT_TOK][X]
-  float* gms = zs + RT_TOK * X;        // [RT_TOK][n_groups] group maxima, then [RT_TOK][n_groups] "may compete" flags
+  float* gms = zs + RT_TOK * X;        // [RT_TOK][n_groups] group scores, then [RT_TOK][n_groups] "may compete" flags
+  float* sgs = gms + 2 * RT_TOK * n_groups;   // [RT_TOK][X] sigmoid scores without the correction (SCORE_SIGMOID only)
   const int m0 = blockIdx.x * RT_TOK;
   const int nt = min(RT_TOK, M - m0);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -83,7 +89,15 @@ __global__ void __launch_bounds__(RT_THREADS) moe_route_kernel(const T* __restri
     const int m = m0 + warp;
     float v0 = 0.f, denom = 0.f;
     float zmax = -INFINITY, zsum = 1.f;
-    if (score_all) {                   // softmax over every expert, also those that cannot be chosen
+    float* sg = sgs + warp * X;
+    if (score == SCORE_SIGMOID) {      // z becomes the choice score
+      for (int e = lane; e < X; e += 32) {
+        sg[e] = 1.f / (1.f + expf(-z[e]));
+        z[e] = sg[e] + (correction ? correction[e] : 0.f);
+      }
+      __syncwarp();
+    }
+    if (score == SCORE_ALL) {          // softmax over every expert, also those that cannot be chosen
       for (int e = lane; e < X; e += 32) zmax = fmaxf(zmax, z[e]);
       zmax = warp_max(zmax);
       float acc = 0.f;
@@ -95,9 +109,12 @@ __global__ void __launch_bounds__(RT_THREADS) moe_route_kernel(const T* __restri
       float* ga = gms + RT_TOK * n_groups + warp * n_groups;
       const int gs = X / n_groups;
       for (int g = lane; g < n_groups; g += 32) {
-        float mx = -INFINITY;
-        for (int e = g * gs; e < (g + 1) * gs; ++e) mx = fmaxf(mx, z[e]);
-        gm[g] = mx;
+        float mx = -INFINITY, m2 = -INFINITY;
+        for (int e = g * gs; e < (g + 1) * gs; ++e) {
+          m2 = fmaxf(m2, fminf(mx, z[e]));
+          mx = fmaxf(mx, z[e]);
+        }
+        gm[g] = group_top == 2 && gs > 1 ? mx + m2 : mx;
       }
       __syncwarp();
       for (int g = lane; g < n_groups; g += 32) {      // a group competes when fewer than keep_groups groups beat it
@@ -124,7 +141,7 @@ __global__ void __launch_bounds__(RT_THREADS) moe_route_kernel(const T* __restri
         if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
       }
       if (k == 0) v0 = best;
-      const float p = score_all ? expf(best - zmax) / zsum : expf(best - v0);
+      const float p = score == SCORE_SIGMOID ? sg[bi] : score == SCORE_ALL ? expf(best - zmax) / zsum : expf(best - v0);
       denom += p;
       if (lane == 0) {
         z[bi] = -INFINITY;
@@ -135,8 +152,8 @@ __global__ void __launch_bounds__(RT_THREADS) moe_route_kernel(const T* __restri
       __syncwarp();
     }
     __syncwarp();
-    if (score_all) denom += 1e-20f;
-    for (int k = lane; k < top; k += 32) expert_w[(size_t)m * top + k] /= denom;
+    if (score != SCORE_CHOSEN) denom += 1e-20f;
+    for (int k = lane; k < top; k += 32) expert_w[(size_t)m * top + k] = expert_w[(size_t)m * top + k] / denom * out_scale;
   }
 }
 
@@ -157,7 +174,7 @@ __global__ void moe_permute_kernel(const int32_t* __restrict__ expert_idx, const
 }
 
 constexpr int GG_BN = 64, GG_BK = 16, GG_THREADS = 256;
-enum { MODE_DOWN = 0, MODE_GLU = 1 };
+enum { MODE_DOWN = 0, MODE_GLU = 1, MODE_RELU2 = 3 };     // (2: MODE_GLU without the shift of the up branch)
 
 // One block = a tile of 16*TM sorted rows of ONE expert x 64 output columns.  fp32 FMAs on operands
 // converted from T (exact for bf16), fp32 accumulation.
@@ -181,8 +198,8 @@ __global__ void __launch_bounds__(GG_THREADS) moe_grouped_gemm_kernel(const T* _
   if (tid < BM) {
     const int r = r0 + min(tid, cnt - 1);
     const int pr = perm[r];
-    src_row[tid] = MODE == MODE_GLU ? pr / top : r;
-    dst_row[tid] = MODE == MODE_GLU ? r : pr;
+    src_row[tid] = MODE != MODE_DOWN ? pr / top : r;
+    dst_row[tid] = MODE != MODE_DOWN ? r : pr;
   }
   __syncthreads();
   const size_t rows_w = MODE == MODE_GLU ? 2 * (size_t)N : (size_t)N;   // rows of one expert's weight
@@ -241,6 +258,7 @@ __global__ void __launch_bounds__(GG_THREADS) moe_grouped_gemm_kernel(const T* _
         v = g / (1.f + expf(-alpha * g)) * (u + shift);
       } else {
         v = acc[0][i][j];
+        if (MODE == MODE_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
       }
       dt<T>::st(c, (size_t)dst_row[r] * ldc + col, v);
     }
@@ -290,8 +308,8 @@ __global__ void __launch_bounds__(GM_THREADS) moe_grouped_gemm_mma_kernel(
   for (int i = tid; i < BM; i += GM_THREADS) {
     const int r = r0 + min(i, cnt - 1);
     const int pr = perm[r];
-    src_row[i] = MODE == MODE_GLU ? pr / top : r;
-    dst_row[i] = MODE == MODE_GLU ? r : pr;
+    src_row[i] = MODE != MODE_DOWN ? pr / top : r;
+    dst_row[i] = MODE != MODE_DOWN ? r : pr;
   }
   __syncthreads();
   const __nv_bfloat16* we = w + (size_t)e * NB * N * K;
@@ -372,6 +390,7 @@ __global__ void __launch_bounds__(GM_THREADS) moe_grouped_gemm_mma_kernel(
           v = g / (1.f + expf(-alpha * g)) * (u + shift);
         } else {
           v = acc[0][i][j][q];
+          if (MODE == MODE_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
         }
         c[(size_t)dst_row[r] * ldc + col] = __float2bfloat16_rn(v);
       }
@@ -420,6 +439,11 @@ static int launch_grouped(const void* a, int lda, const void* w, const int32_t* 
   return LL_OK;
 }
 
+template <int TM, int MODE, typename... A>
+static int launch_grouped_f32(A... args) { return launch_grouped<float, TM, MODE>(args...); }
+template <int TM, int MODE, typename... A>
+static int launch_grouped_bf16(A... args) { return launch_grouped<__nv_bfloat16, TM, MODE>(args...); }
+
 }  // namespace llb
 
 using namespace llb;
@@ -436,33 +460,44 @@ int ll_moe_route(const void* x, int dtype, const float* w_router, const float* b
 int ll_moe_route_scored(const void* x, int dtype, const float* w_router, const float* bias, int M, int dim, int n_experts, int top,
                         int score_all, int n_groups, int keep_groups, int32_t* expert_idx, float* expert_w, int32_t* counts,
                         int32_t* rank, int32_t* offsets, int32_t* perm, ll_stream stream) {
+  return ll_moe_route_choice(x, dtype, w_router, bias, M, dim, n_experts, top, score_all ? SCORE_ALL : SCORE_CHOSEN, nullptr, 1.f, n_groups,
+                             keep_groups, 1, expert_idx, expert_w, counts, rank, offsets, perm, stream);
+}
+
+int ll_moe_route_choice(const void* x, int dtype, const float* w_router, const float* bias, int M, int dim, int n_experts, int top,
+                        int score, const float* correction, float out_scale, int n_groups, int keep_groups, int group_top,
+                        int32_t* expert_idx, float* expert_w, int32_t* counts, int32_t* rank, int32_t* offsets, int32_t* perm,
+                        ll_stream stream) {
   LL_CHECK_ARG(x && w_router && expert_idx && expert_w && counts && rank && offsets && perm, "moe_route: null pointer");
   LL_CHECK_ARG(M >= 0 && dim > 0 && n_experts > 0 && top > 0 && top <= n_experts, "bad moe_route arguments");
+  LL_CHECK_ARG(score >= SCORE_CHOSEN && score <= SCORE_SIGMOID && (!correction || score == SCORE_SIGMOID) && (group_top == 1 || group_top == 2),
+               "moe_route: score %d, group score of %d", score, group_top);
   LL_CHECK_ARG(n_groups >= 1 && keep_groups >= 1 && keep_groups <= n_groups && n_experts % n_groups == 0 &&
                    top <= keep_groups * (n_experts / n_groups),
                "moe_route: %d groups (keep %d) of %d experts cannot give %d choices", n_groups, keep_groups, n_experts, top);
   if (M == 0) return LL_OK;
   cudaStream_t st = (cudaStream_t)stream;
-  const size_t smem = sizeof(float) * RT_TOK * ((size_t)dim + n_experts + 2 * (size_t)n_groups);
+  const size_t smem =
+      sizeof(float) * RT_TOK * ((size_t)dim + (score == SCORE_SIGMOID ? 2 : 1) * (size_t)n_experts + 2 * (size_t)n_groups);
   if (smem > 200 * 1024) {
     set_error("moe_route: width %d with %d experts does not fit shared memory", dim, n_experts);
     return LL_ERR_UNSUPPORTED;
   }
   LL_CUDA(cudaMemsetAsync(counts, 0, sizeof(int32_t) * n_experts, st));
   const int blocks = (M + RT_TOK - 1) / RT_TOK;
+#define LL_RT(T)                                                                                                                     \
+  LL_CUDA(cudaFuncSetAttribute(moe_route_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));                       \
+  moe_route_kernel<T><<<blocks, RT_THREADS, smem, st>>>((const T*)x, w_router, bias, M, dim, n_experts, top, score, correction, out_scale, \
+                                                        n_groups, keep_groups, group_top, expert_idx, expert_w, counts, rank)
   if (dtype == LL_F32) {
-    LL_CUDA(cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    moe_route_kernel<float><<<blocks, RT_THREADS, smem, st>>>((const float*)x, w_router, bias, M, dim, n_experts, top, score_all,
-                                                             n_groups, keep_groups, expert_idx, expert_w, counts, rank);
+    LL_RT(float);
   } else if (dtype == LL_BF16) {
-    LL_CUDA(cudaFuncSetAttribute(moe_route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    moe_route_kernel<__nv_bfloat16><<<blocks, RT_THREADS, smem, st>>>((const __nv_bfloat16*)x, w_router, bias, M, dim, n_experts, top,
-                                                                     score_all, n_groups, keep_groups, expert_idx, expert_w, counts,
-                                                                     rank);
+    LL_RT(__nv_bfloat16);
   } else {
     set_error("moe_route: unsupported dtype %d", dtype);
     return LL_ERR_UNSUPPORTED;
   }
+#undef LL_RT
   LL_LAUNCH_OK("moe_route_kernel");
   const int n_pairs = M * top;
   moe_permute_kernel<<<(n_pairs + 255) / 256, 256, sizeof(int32_t) * (n_experts + 1), st>>>(expert_idx, rank, counts, n_pairs,
@@ -475,28 +510,27 @@ int ll_moe_grouped_gemm(const void* a, int lda, const void* w, const int32_t* of
                         int n_rows, int top, int n_experts, int N, int K, float limit, float alpha, void* c, int ldc,
                         ll_stream stream) {
   LL_CHECK_ARG(a && w && offsets && perm && c, "moe_grouped_gemm: null pointer");
-  LL_CHECK_ARG(n_rows >= 0 && top > 0 && n_experts > 0 && N > 0 && K > 0 && lda >= K && ldc >= N && mode >= 0 && mode <= 2,
+  LL_CHECK_ARG(n_rows >= 0 && top > 0 && n_experts > 0 && N > 0 && K > 0 && lda >= K && ldc >= N && mode >= 0 && mode <= 3,
                "bad moe_grouped_gemm arguments");
   if (n_rows == 0) return LL_OK;
   const float shift = mode == 2 ? 0.f : 1.f;     // mode 2: the up branch enters as it is
   if (mode == 2) mode = MODE_GLU;
   cudaStream_t st = (cudaStream_t)stream;
   const bool small = n_rows <= 16 * n_experts / 2 + 16;   // few rows per expert: narrow row tiles waste less
-#define LL_GG(T)                                                                                                              \
-  (mode == MODE_GLU ? (small ? launch_grouped<T, 1, MODE_GLU>(a, lda, w, offsets, perm, top, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st)  \
-                             : launch_grouped<T, 4, MODE_GLU>(a, lda, w, offsets, perm, top, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st)) \
-                    : (small ? launch_grouped<T, 1, MODE_DOWN>(a, lda, w, offsets, perm, top, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st) \
-                             : launch_grouped<T, 4, MODE_DOWN>(a, lda, w, offsets, perm, top, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st)))
-  if (dtype == LL_F32) return LL_GG(float);
+#define LL_GG_MODE(FN, NARROW, WIDE, MODE)                                                                                          \
+  return small ? FN<NARROW, MODE>(a, lda, w, offsets, perm, top, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st)            \
+               : FN<WIDE, MODE>(a, lda, w, offsets, perm, top, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st)
+#define LL_GG(FN, NARROW, WIDE)                                  \
+  if (mode == MODE_GLU) LL_GG_MODE(FN, NARROW, WIDE, MODE_GLU);  \
+  if (mode == MODE_RELU2) LL_GG_MODE(FN, NARROW, WIDE, MODE_RELU2); \
+  LL_GG_MODE(FN, NARROW, WIDE, MODE_DOWN)
+  if (dtype == LL_F32) { LL_GG(launch_grouped_f32, 1, 4); }
   if (dtype == LL_BF16 && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)a & 15) == 0 && ((uintptr_t)w & 15) == 0) {
-    if (mode == MODE_GLU)
-      return small ? launch_grouped_mma<16, MODE_GLU>(a, lda, w, offsets, perm, top, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st)
-                   : launch_grouped_mma<64, MODE_GLU>(a, lda, w, offsets, perm, top, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st);
-    return small ? launch_grouped_mma<16, MODE_DOWN>(a, lda, w, offsets, perm, top, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st)
-                 : launch_grouped_mma<64, MODE_DOWN>(a, lda, w, offsets, perm, top, n_experts, N, K, limit, alpha, shift, c, ldc, n_rows, st);
+    LL_GG(launch_grouped_mma, 16, 64);
   }
-  if (dtype == LL_BF16) return LL_GG(__nv_bfloat16);
+  if (dtype == LL_BF16) { LL_GG(launch_grouped_bf16, 1, 4); }
 #undef LL_GG
+#undef LL_GG_MODE
   set_error("moe_grouped_gemm: unsupported dtype %d", dtype);
   return LL_ERR_UNSUPPORTED;
 }

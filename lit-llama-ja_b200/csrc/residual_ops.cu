@@ -70,19 +70,76 @@ __global__ void gain_norm_add_mix_kernel(const float* x, const TY* __restrict__ 
   }
 }
 
+// Eight neighbouring numbers of an activation row as fp32 (16-byte accesses in bf16, two in fp32).
+template <typename T> __device__ __forceinline__ void ld8(const T* p, float (&o)[8]);
+template <> __device__ __forceinline__ void ld8<float>(const float* p, float (&o)[8]) {
+  const float4 a = ((const float4*)p)[0], b = ((const float4*)p)[1];
+  o[0] = a.x, o[1] = a.y, o[2] = a.z, o[3] = a.w, o[4] = b.x, o[5] = b.y, o[6] = b.z, o[7] = b.w;
+}
+template <> __device__ __forceinline__ void ld8<__nv_bfloat16>(const __nv_bfloat16* p, float (&o)[8]) {
+  const uint4 u = *(const uint4*)p;
+  o[0] = bf16_bits_to_f32(u.x & 0xffffu), o[1] = bf16_bits_to_f32(u.x >> 16);
+  o[2] = bf16_bits_to_f32(u.y & 0xffffu), o[3] = bf16_bits_to_f32(u.y >> 16);
+  o[4] = bf16_bits_to_f32(u.z & 0xffffu), o[5] = bf16_bits_to_f32(u.z >> 16);
+  o[6] = bf16_bits_to_f32(u.w & 0xffffu), o[7] = bf16_bits_to_f32(u.w >> 16);
+}
+template <typename T> __device__ __forceinline__ void st8(T* p, const float (&v)[8]);
+template <> __device__ __forceinline__ void st8<float>(float* p, const float (&v)[8]) {
+  ((float4*)p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+  ((float4*)p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+template <> __device__ __forceinline__ void st8<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[8]) {
+  uint32_t k[4];
+#pragma unroll
+  for (int q = 0; q < 4; ++q) k[q] = (uint32_t)f32_to_bf16_bits(v[2 * q]) | ((uint32_t)f32_to_bf16_bits(v[2 * q + 1]) << 16);
+  *(uint4*)p = make_uint4(k[0], k[1], k[2], k[3]);
+}
+
 // Gated linear unit with clamped pre-activations, on the output of one GEMM over the stacked
 // [gate; up] weight:  g = min(gu[m][c], limit), u = clamp(gu[m][ff + c], -limit, limit),
-// h[m][c] = g * sigmoid(alpha * g) * (u + 1).
+// h[m][c] = g * sigmoid(alpha * g) * (u + shift).
+__device__ __forceinline__ float glu_unit(float g, float u, float limit, float alpha, float shift) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g / (1.f + expf(-alpha * g)) * (u + shift);
+}
 template <typename T>
-__global__ void glu_clamp_kernel(const T* __restrict__ gu, int gu_stride, int ff, float limit, float alpha,
-                                 T* __restrict__ h, size_t n) {
+__global__ void glu_unit_kernel(const T* __restrict__ gu, int gu_stride, int ff, float limit, float alpha, float shift,
+                                T* __restrict__ h, size_t n) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n) return;
   const size_t m = i / ff;
   const int c = (int)(i - m * ff);
-  const float g = fminf(dt<T>::ld(gu, m * gu_stride + c), limit);
-  const float u = fminf(fmaxf(dt<T>::ld(gu, m * gu_stride + ff + c), -limit), limit);
-  dt<T>::st(h, i, g / (1.f + expf(-alpha * g)) * (u + 1.f));
+  dt<T>::st(h, i, glu_unit(dt<T>::ld(gu, m * gu_stride + c), dt<T>::ld(gu, m * gu_stride + ff + c), limit, alpha, shift));
+}
+// ff, gu_stride multiples of 8 and 16-byte aligned rows: a thread owns eight columns of one row
+template <typename T>
+__global__ void glu_unit8_kernel(const T* __restrict__ gu, int gu_stride, int ff, float limit, float alpha, float shift,
+                                 T* __restrict__ h, int n8) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n8) return;
+  const int per = ff / 8, m = i / per, c = (i - m * per) * 8;
+  const T* row = gu + (size_t)m * gu_stride + c;
+  float g[8], u[8];
+  ld8<T>(row, g);
+  ld8<T>(row + ff, u);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) g[e] = glu_unit(g[e], u[e], limit, alpha, shift);
+  st8<T>(h + (size_t)m * ff + c, g);
+}
+
+template <typename T>
+static int glu_unit_launch(const void* gu, int gu_stride, int ff, float limit, float alpha, float shift, void* h, int rows,
+                           cudaStream_t st) {
+  const size_t n = (size_t)rows * ff;
+  if (ff % 8 == 0 && gu_stride % 8 == 0 && (((uintptr_t)gu | (uintptr_t)h) & 15) == 0 && n / 8 < (1ull << 31)) {
+    const int n8 = (int)(n / 8);
+    glu_unit8_kernel<T><<<(n8 + 127) / 128, 128, 0, st>>>((const T*)gu, gu_stride, ff, limit, alpha, shift, (T*)h, n8);
+  } else {
+    glu_unit_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, st>>>((const T*)gu, gu_stride, ff, limit, alpha, shift, (T*)h, n);
+  }
+  LL_LAUNCH_OK("glu_unit_kernel");
+  return LL_OK;
 }
 
 }  // namespace llb
@@ -138,22 +195,20 @@ int ll_gain_norm_add_mix(const float* x, const void* y, int y_dtype, const float
   return LL_OK;
 }
 
+int ll_glu_unit(const void* gu, int gu_stride, int ff, float limit, float alpha, float shift, void* h, int dtype, int rows,
+                ll_stream stream) {
+  LL_CHECK_ARG(gu && h && ff > 0 && gu_stride >= 2 * ff && rows >= 0, "bad glu_unit arguments");
+  if (rows == 0) return LL_OK;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (dtype == LL_F32) return glu_unit_launch<float>(gu, gu_stride, ff, limit, alpha, shift, h, rows, st);
+  if (dtype == LL_BF16) return glu_unit_launch<__nv_bfloat16>(gu, gu_stride, ff, limit, alpha, shift, h, rows, st);
+  set_error("glu_unit: unsupported dtype %d", dtype);
+  return LL_ERR_UNSUPPORTED;
+}
+
 int ll_glu_clamp(const void* gu, int gu_stride, int ff, float limit, float alpha, void* h, int dtype, int rows,
                  ll_stream stream) {
-  LL_CHECK_ARG(gu && h && ff > 0 && gu_stride >= 2 * ff && rows >= 0, "bad glu_clamp arguments");
-  const size_t n = (size_t)rows * ff;
-  if (n == 0) return LL_OK;
-  cudaStream_t st = (cudaStream_t)stream;
-  const unsigned blocks = (unsigned)((n + 255) / 256);
-  if (dtype == LL_F32) glu_clamp_kernel<float><<<blocks, 256, 0, st>>>((const float*)gu, gu_stride, ff, limit, alpha, (float*)h, n);
-  else if (dtype == LL_BF16)
-    glu_clamp_kernel<__nv_bfloat16><<<blocks, 256, 0, st>>>((const __nv_bfloat16*)gu, gu_stride, ff, limit, alpha, (__nv_bfloat16*)h, n);
-  else {
-    set_error("glu_clamp: unsupported dtype %d", dtype);
-    return LL_ERR_UNSUPPORTED;
-  }
-  LL_LAUNCH_OK("glu_clamp_kernel");
-  return LL_OK;
+  return ll_glu_unit(gu, gu_stride, ff, limit, alpha, 1.f, h, dtype, rows, stream);
 }
 
 }  // extern "C"
@@ -194,6 +249,116 @@ __global__ void add_norm_pair_kernel(float* __restrict__ x, const TA* __restrict
     }
     if (out2) dt<TA>::st(out2, base + i, n * w2[i]);
   }
+}
+
+// x[m][:] += s * a (optional, activation dtype TA), in place, fp32.  Then, if asked for, the layer norm of the same row:
+// out = (x - mean) / sqrt(var + eps) * w + b, var the mean of the squared deviations (formed from the deviations themselves,
+// in a second sweep over the row the block holds).  One block per row; VPT > 0: the row stays in registers, VPT runs of four
+// numbers per thread; VPT = 0: any length, the row in shared memory.
+template <typename TA> __device__ __forceinline__ float4 ld4(const TA* p);
+template <> __device__ __forceinline__ float4 ld4<float>(const float* p) { return *(const float4*)p; }
+template <> __device__ __forceinline__ float4 ld4<__nv_bfloat16>(const __nv_bfloat16* p) {
+  const uint2 u = *(const uint2*)p;
+  return make_float4(bf16_bits_to_f32(u.x & 0xffffu), bf16_bits_to_f32(u.x >> 16), bf16_bits_to_f32(u.y & 0xffffu),
+                     bf16_bits_to_f32(u.y >> 16));
+}
+template <typename TA> __device__ __forceinline__ void st4(TA* p, float4 v);
+template <> __device__ __forceinline__ void st4<float>(float* p, float4 v) { *(float4*)p = v; }
+template <> __device__ __forceinline__ void st4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+  *(uint2*)p = make_uint2((uint32_t)f32_to_bf16_bits(v.x) | ((uint32_t)f32_to_bf16_bits(v.y) << 16),
+                          (uint32_t)f32_to_bf16_bits(v.z) | ((uint32_t)f32_to_bf16_bits(v.w) << 16));
+}
+
+template <typename TA, int VPT>
+__global__ void add_layer_norm_kernel(float* __restrict__ x, const TA* __restrict__ a, float s, const float* __restrict__ w,
+                                      const float* __restrict__ b, float eps, TA* __restrict__ out, int dim) {
+  extern __shared__ float ln_row[];
+  __shared__ float red[32];
+  const size_t base = (size_t)blockIdx.x * dim;
+  float sum = 0.f;
+  if constexpr (VPT > 0) {
+    float4 v[VPT > 0 ? VPT : 1], av[VPT > 0 ? VPT : 1];
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 4;
+      v[k] = i < dim ? *(const float4*)(x + base + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      if (a) av[k] = i < dim ? ld4<TA>(a + base + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 4;
+      if (a) {
+        v[k].x += s * av[k].x, v[k].y += s * av[k].y, v[k].z += s * av[k].z, v[k].w += s * av[k].w;
+        if (i < dim) *(float4*)(x + base + i) = v[k];
+      }
+      sum += (v[k].x + v[k].y) + (v[k].z + v[k].w);
+    }
+    if (!out) return;
+    const float mean = block_sum(sum, red) / (float)dim;
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 4;
+      v[k].x -= mean, v[k].y -= mean, v[k].z -= mean, v[k].w -= mean;
+      if (i < dim) ss += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+    }
+    const float kn = 1.f / sqrtf(block_sum(ss, red) / (float)dim + eps);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 4;
+      if (i < dim) {
+        const float4 wv = *(const float4*)(w + i), bv = *(const float4*)(b + i);
+        st4<TA>(out + base + i, make_float4(v[k].x * kn * wv.x + bv.x, v[k].y * kn * wv.y + bv.y, v[k].z * kn * wv.z + bv.z,
+                                            v[k].w * kn * wv.w + bv.w));
+      }
+    }
+  } else {
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) {
+      float v = x[base + i];
+      if (a) {
+        v += s * dt<TA>::ld(a, base + i);
+        x[base + i] = v;
+      }
+      ln_row[i] = v;
+      sum += v;
+    }
+    if (!out) return;
+    const float mean = block_sum(sum, red) / (float)dim;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) {      // (a thread reads back what it wrote itself)
+      const float d = ln_row[i] - mean;
+      ss += d * d;
+    }
+    const float kn = 1.f / sqrtf(block_sum(ss, red) / (float)dim + eps);
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) dt<TA>::st(out, base + i, (ln_row[i] - mean) * kn * w[i] + b[i]);
+  }
+}
+
+template <typename TA>
+static int add_layer_norm_launch(float* x, const void* a, float s, const float* w, const float* b, float eps, void* out, int rows, int dim,
+                                 cudaStream_t st) {
+  const bool vec = dim % 4 == 0 && dim <= 8192 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)a | (uintptr_t)out) & 15) == 0;
+#define LL_ALN(VPT, NT, SM) add_layer_norm_kernel<TA, VPT><<<rows, NT, SM, st>>>(x, (const TA*)a, s, w, b, eps, (TA*)out, dim)
+  if (vec) {
+    if (dim <= 2048) LL_ALN(1, (dim / 4 + 31) / 32 * 32, 0);
+    else if (dim <= 4096) LL_ALN(2, 512, 0);
+    else LL_ALN(4, 512, 0);
+  } else {
+    const size_t smem = (size_t)dim * sizeof(float);
+    if (smem > 200 * 1024) {
+      set_error("add_layer_norm: rows of %d numbers", dim);
+      return LL_ERR_UNSUPPORTED;
+    }
+    static bool sized = false;
+    if (!sized && smem > 48 * 1024) {
+      LL_CUDA(cudaFuncSetAttribute(add_layer_norm_kernel<TA, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+      sized = true;
+    }
+    LL_ALN(0, dim >= 512 ? 256 : 128, smem);
+  }
+#undef LL_ALN
+  LL_LAUNCH_OK("add_layer_norm_kernel");
+  return LL_OK;
 }
 
 // RMS norm of an fp32 row in `groups` equal parts (each by its own root mean square), a weight, and a gate (silu, or a
@@ -237,6 +402,30 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, int y_gs, c
   }
 }
 
+// The same for long parts (a whole row of heads normed together): a block per (row, part), the gated numbers of the first sweep
+// kept in shared memory.
+template <typename TA>
+__global__ void gated_group_norm_wide_kernel(const float* __restrict__ y, const TA* __restrict__ gate, int gate_stride,
+                                             const float* __restrict__ w, int w_shared, float eps, int gate_first, int gate_sigmoid,
+                                             TA* __restrict__ out, int gs) {
+  extern __shared__ float ggn_row[];
+  __shared__ float red[32];
+  const size_t m = blockIdx.y;
+  const int g = blockIdx.x, groups = gridDim.x;
+  const float* yr = y + (m * groups + g) * gs;
+  const TA* gr = gate + m * gate_stride + (size_t)g * gs;
+  const float* wr = w + (w_shared ? 0 : (size_t)g * gs);
+  TA* orow = out + (m * groups + g) * gs;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < gs; i += blockDim.x) {
+    const float z = dt<TA>::ld(gr, i), sg = (gate_sigmoid ? 1.f : z) / (1.f + expf(-z)), v = yr[i];
+    ss += gate_first ? (v * sg) * (v * sg) : v * v;
+    ggn_row[i] = v * sg;
+  }
+  const float k = 1.f / sqrtf(block_sum(ss, red) / (float)gs + eps);
+  for (int i = threadIdx.x; i < gs; i += blockDim.x) dt<TA>::st(orow, i, ggn_row[i] * k * wr[i]);
+}
+
 // in place: relu(v)^2
 template <typename T>
 __global__ void relu_squared_kernel(T* __restrict__ h, size_t n) {
@@ -244,6 +433,20 @@ __global__ void relu_squared_kernel(T* __restrict__ h, size_t n) {
   if (i >= n) return;
   const float v = fmaxf(dt<T>::ld(h, i), 0.f);
   dt<T>::st(h, i, v * v);
+}
+
+template <typename T>
+__global__ void relu_squared8_kernel(T* __restrict__ h, size_t n8) {
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n8) return;
+  float v[8];
+  ld8<T>(h + i * 8, v);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    const float r = fmaxf(v[e], 0.f);
+    v[e] = r * r;
+  }
+  st8<T>(h + i * 8, v);
 }
 
 // in place: gelu(v), the erf form 0.5 v (1 + erf(v / sqrt 2)) or (tanh_form) 0.5 v (1 + tanh(sqrt(2/pi) (v + 0.044715 v^3)))
@@ -469,6 +672,17 @@ int ll_add_norm_pair(float* x, const void* a0, float s0, const void* a1, float s
   return LL_OK;
 }
 
+int ll_add_layer_norm(float* x, const void* a, float s, const float* w, const float* b, float eps, void* out, int act_dtype, int rows,
+                      int dim, ll_stream stream) {
+  LL_CHECK_ARG(x && rows >= 0 && dim > 0 && (!out || (w && b)), "bad add_layer_norm arguments");
+  if (rows == 0) return LL_OK;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (act_dtype == LL_F32) return add_layer_norm_launch<float>(x, a, s, w, b, eps, out, rows, dim, st);
+  if (act_dtype == LL_BF16) return add_layer_norm_launch<__nv_bfloat16>(x, a, s, w, b, eps, out, rows, dim, st);
+  set_error("add_layer_norm: unsupported dtype %d", act_dtype);
+  return LL_ERR_UNSUPPORTED;
+}
+
 int ll_gated_group_norm(const float* y, int y_gs, const float* stab, const void* gate, int gate_stride, const float* w, int w_shared,
                         float eps, int groups, int gate_first, int gate_sigmoid, void* out, int act_dtype, int rows, int C,
                         ll_stream stream) {
@@ -478,6 +692,23 @@ int ll_gated_group_norm(const float* y, int y_gs, const float* stab, const void*
   LL_CHECK_ARG(y_gs >= C / groups + (stab ? 1 : 0), "gated_group_norm: a part of y is shorter than the part it norms");
   if (rows == 0) return LL_OK;
   cudaStream_t st = (cudaStream_t)stream;
+  const int gs = C / groups;
+  if (gs >= 256 && gs <= 12288 && !stab && y_gs == gs && rows <= 65535) {
+    const int nt = gs >= 1024 ? 256 : 128;
+    const size_t smem = (size_t)gs * sizeof(float);
+    if (act_dtype == LL_F32)
+      gated_group_norm_wide_kernel<float><<<dim3(groups, rows), nt, smem, st>>>(y, (const float*)gate, gate_stride, w, w_shared, eps,
+                                                                               gate_first, gate_sigmoid, (float*)out, gs);
+    else if (act_dtype == LL_BF16)
+      gated_group_norm_wide_kernel<__nv_bfloat16><<<dim3(groups, rows), nt, smem, st>>>(
+          y, (const __nv_bfloat16*)gate, gate_stride, w, w_shared, eps, gate_first, gate_sigmoid, (__nv_bfloat16*)out, gs);
+    else {
+      set_error("gated_group_norm: unsupported dtype %d", act_dtype);
+      return LL_ERR_UNSUPPORTED;
+    }
+    LL_LAUNCH_OK("gated_group_norm_wide_kernel");
+    return LL_OK;
+  }
   const int threads = groups >= 8 ? 256 : groups >= 4 ? 128 : 32 * groups;
   if (act_dtype == LL_F32)
     gated_group_norm_kernel<float><<<rows, threads, 0, st>>>(y, y_gs, stab, (const float*)gate, gate_stride, w, w_shared, eps, groups,
@@ -498,7 +729,11 @@ int ll_relu_squared(void* h, int dtype, size_t n, ll_stream stream) {
   if (n == 0) return LL_OK;
   cudaStream_t st = (cudaStream_t)stream;
   const unsigned blocks = (unsigned)((n + 255) / 256);
-  if (dtype == LL_F32) relu_squared_kernel<float><<<blocks, 256, 0, st>>>((float*)h, n);
+  const bool vec = n % 8 == 0 && ((uintptr_t)h & 15) == 0;
+  const unsigned blocks8 = (unsigned)((n / 8 + 127) / 128);
+  if (dtype == LL_F32 && vec) relu_squared8_kernel<float><<<blocks8, 128, 0, st>>>((float*)h, n / 8);
+  else if (dtype == LL_BF16 && vec) relu_squared8_kernel<__nv_bfloat16><<<blocks8, 128, 0, st>>>((__nv_bfloat16*)h, n / 8);
+  else if (dtype == LL_F32) relu_squared_kernel<float><<<blocks, 256, 0, st>>>((float*)h, n);
   else if (dtype == LL_BF16) relu_squared_kernel<__nv_bfloat16><<<blocks, 256, 0, st>>>((__nv_bfloat16*)h, n);
   else {
     set_error("relu_squared: unsupported dtype %d", dtype);

@@ -3,7 +3,10 @@
 //   prepare   q, k <- [rmsnorm over the WHOLE projection row * w]  ->  rotation of the first `rot_dims` dimensions of every head
 //             (dimension i paired with i + rot_dims/2, angle = position * freq[i], all fp32)  ->  q rows out, k rows into the
 //             ring at slot position % ring; the value rows are a projection of their own or the keys BEFORE rotation.
-//   attend    s_h(i, j) = scale * q_h(i).k_g(j),  optionally cap * tanh(s / cap);
+//             Or, with a norm per HEAD (one weight of the head's size for all heads): every head of q and k divided by its own
+//             root mean square, the queries optionally times 1 + coef * ln(floor((position + 1) / every) + 1), the values
+//             optionally mixed with another layer's values of the same token.
+//   attend    s_h(i, j) = scale * q_h(i).k_g(j),  optionally minus slope_h * (i - j),  optionally cap * tanh(s / cap);
 //             key j visible to query i when j <= i, (window == 0 or i - j < window), (chunk == 0 or j / chunk == i / chunk);
 //             softmax over the visible keys, optionally with exp(sink_h) added to the denominator (a key without a value);
 //             o_h(i) = sum_j w(i, j) v_g(j), optionally times sigmoid(gate) element by element.
@@ -93,6 +96,124 @@ __global__ void __launch_bounds__(QP_THREADS) qk_rotary_append_kernel(
     for (int i = threadIdx.x; i < G * vdim; i += blockDim.x) vrow[i] = v[(size_t)m * v_stride + i];
 }
 
+// Heads of a row normed one by one: a warp owns a head, its numbers pass through the warp's shared row (the rotation pairs
+// distant dimensions).  q heads, then k heads, then the values element by element over the whole block.
+constexpr int QH_WARPS = QP_THREADS / 32, QH_DIM = 256;
+
+template <typename T>
+__device__ __forceinline__ void qh_load2(const T* p, int i, int n, bool pair, float& a, float& b) {
+  a = i < n ? dt<T>::ld(p, i) : 0.f;
+  b = i + 1 < n ? dt<T>::ld(p, i + 1) : 0.f;
+}
+template <>
+__device__ __forceinline__ void qh_load2<__nv_bfloat16>(const __nv_bfloat16* p, int i, int n, bool pair, float& a, float& b) {
+  if (pair && i + 1 < n) {
+    const uint32_t u = *(const uint32_t*)(p + i);
+    a = bf16_bits_to_f32(u & 0xffffu), b = bf16_bits_to_f32(u >> 16);
+  } else {
+    a = i < n ? __bfloat162float(p[i]) : 0.f;
+    b = i + 1 < n ? __bfloat162float(p[i + 1]) : 0.f;
+  }
+}
+template <typename T>
+__device__ __forceinline__ void qh_store2(T* p, int i, int n, bool pair, float a, float b) {
+  if (i < n) dt<T>::st(p, i, a);
+  if (i + 1 < n) dt<T>::st(p, i + 1, b);
+}
+template <>
+__device__ __forceinline__ void qh_store2<__nv_bfloat16>(__nv_bfloat16* p, int i, int n, bool pair, float a, float b) {
+  if (pair && i + 1 < n) {
+    *(uint32_t*)(p + i) = (uint32_t)f32_to_bf16_bits(a) | ((uint32_t)f32_to_bf16_bits(b) << 16);
+  } else {
+    if (i < n) p[i] = __float2bfloat16_rn(a);
+    if (i + 1 < n) p[i + 1] = __float2bfloat16_rn(b);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(QP_THREADS) qk_head_append_kernel(
+    const T* __restrict__ q, int q_stride, const T* __restrict__ k, int k_stride, const T* __restrict__ v, int v_stride,
+    const T* __restrict__ first, int first_stride, float lam, const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps,
+    const float* __restrict__ freq, int rot_dims, float temp_coef, int temp_every, const int32_t* __restrict__ pos_ids,
+    T* __restrict__ q_out, T* __restrict__ kc, T* __restrict__ vc, int Tn, int H, int G, int dim, int vdim, int ring, int pair) {
+  __shared__ float row[QH_WARPS][QH_DIM];
+  const int m = blockIdx.x, b = m / Tn, t = m - b * Tn;
+  const int p = pos_ids[t], warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = rot_dims >> 1;
+  const float temp = temp_every > 0 ? 1.f + temp_coef * logf((float)((p + 1) / temp_every) + 1.f) : 1.f;
+  const size_t slot = (size_t)b * ring + (size_t)(p % ring);
+  for (int hh = warp; hh < H + G; hh += QH_WARPS) {
+    const bool is_q = hh < H;
+    const T* src = is_q ? q + (size_t)m * q_stride + (size_t)hh * dim : k + (size_t)m * k_stride + (size_t)(hh - H) * dim;
+    T* dst = is_q ? q_out + ((size_t)m * H + hh) * dim : kc + (slot * G + (hh - H)) * dim;
+    const float* nw = is_q ? q_norm : k_norm;
+    float e0[QH_DIM / 64], e1[QH_DIM / 64], ss = 0.f;
+#pragma unroll
+    for (int r = 0; r < QH_DIM / 64; ++r) {
+      const int i = 2 * (lane + 32 * r);
+      if (r * 64 < dim) {
+        qh_load2<T>(src, i, dim, pair, e0[r], e1[r]);
+        ss += e0[r] * e0[r] + e1[r] * e1[r];
+      }
+    }
+    ss = warp_sum(ss);
+    const float kn = nw ? 1.f / sqrtf(ss / (float)dim + eps) : 1.f;
+    const float mult = is_q ? temp : 1.f;
+    if (rot_dims > 0) __syncwarp();              // the row's readers of the head before are done
+#pragma unroll
+    for (int r = 0; r < QH_DIM / 64; ++r) {
+      const int i = 2 * (lane + 32 * r);
+      if (r * 64 < dim) {
+        e0[r] *= kn, e1[r] *= kn;
+        if (nw) {
+          if (i < dim) e0[r] *= nw[i];
+          if (i + 1 < dim) e1[r] *= nw[i + 1];
+        }
+        e0[r] *= mult, e1[r] *= mult;
+        if (rot_dims > 0) {
+          row[warp][i] = e0[r];
+          row[warp][i + 1] = e1[r];
+        }
+      }
+    }
+    if (rot_dims > 0) {
+      __syncwarp();
+#pragma unroll
+      for (int r = 0; r < QH_DIM / 64; ++r) {
+        const int i = 2 * (lane + 32 * r);
+        if (r * 64 < dim) {
+#pragma unroll
+          for (int z = 0; z < 2; ++z) {
+            const int c = i + z;
+            if (c >= rot_dims) continue;
+            const bool lower = c < half;
+            float sn, cs;
+            sincosf((float)p * freq[lower ? c : c - half], &sn, &cs);
+            const float a = row[warp][c], o = row[warp][lower ? c + half : c - half];
+            (z ? e1[r] : e0[r]) = lower ? a * cs - o * sn : a * cs + o * sn;
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < QH_DIM / 64; ++r)
+      if (r * 64 < dim) qh_store2<T>(dst, 2 * (lane + 32 * r), dim, pair, e0[r], e1[r]);
+  }
+  T* vrow = vc + slot * (size_t)G * vdim;
+  const T* vsrc = v + (size_t)m * v_stride;
+  const T* fsrc = first ? first + (size_t)m * first_stride : nullptr;
+  for (int i = 2 * threadIdx.x; i < G * vdim; i += 2 * QP_THREADS) {
+    float a, c;
+    qh_load2<T>(vsrc, i, G * vdim, pair, a, c);
+    if (fsrc) {
+      float fa, fc;
+      qh_load2<T>(fsrc, i, G * vdim, pair, fa, fc);
+      a = (1.f - lam) * a + lam * fa;
+      c = (1.f - lam) * c + lam * fc;
+    }
+    qh_store2<T>(vrow, i, G * vdim, pair, a, c);
+  }
+}
+
 // ---------------------------------------------------------------------------------------------------------------- attend, fp32 form
 // A warp owns one (query, head); its four groups of eight lanes take every fourth visible key, the eight lanes of a group
 // split the head's dimensions in runs of eight (one 16-byte load in bf16).  Every group keeps a running (max, sum, weighted
@@ -144,8 +265,8 @@ __device__ __forceinline__ int sa_first_visible(int i, int window, int chunk) {
 template <typename T, int R, int RV>
 __global__ void __launch_bounds__(SA_WARPS * 32) softmax_attn_kernel(
     const T* __restrict__ q, int q_stride, const T* __restrict__ gate, int gate_stride, const T* __restrict__ kc, const T* __restrict__ vc,
-    const int32_t* __restrict__ pos_ids, const float* __restrict__ sink, float scale, float softcap, int Tn, int H, int G, int dim,
-    int vdim, int window, int chunk, int ring, int splits, int maps, int pairs, float* __restrict__ part_ml,
+    const int32_t* __restrict__ pos_ids, const float* __restrict__ sink, const float* __restrict__ slopes, float scale, float softcap,
+    int Tn, int H, int G, int dim, int vdim, int window, int chunk, int ring, int splits, int maps, int pairs, float* __restrict__ part_ml,
     float* __restrict__ part_acc, T* __restrict__ y) {
   // a warp owns one (query, head, map); with one map per head, h below is the head itself
   const int pair = blockIdx.x * SA_WARPS + (threadIdx.x >> 5);
@@ -172,6 +293,7 @@ __global__ void __launch_bounds__(SA_WARPS * 32) softmax_attn_kernel(
     for (int e = 0; e < 8; ++e) acc[r][e] = 0.f;
   float mx = -INFINITY, l = 0.f;
   const float inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
+  const float slope = slopes ? slopes[head] : 0.f;
   const T* kbase = kc + ((size_t)b * ring * GK + gk) * dim;
   const T* vbase = vc + ((size_t)b * ring * G + g) * vdim;
   const unsigned gmask = 0xffu << (grp * 8);
@@ -190,6 +312,7 @@ __global__ void __launch_bounds__(SA_WARPS * 32) softmax_attn_kernel(
     s += __shfl_xor_sync(gmask, s, 2);
     s += __shfl_xor_sync(gmask, s, 4);
     s *= scale;
+    if (slopes) s -= slope * (float)(i - j);
     if (softcap > 0.f) s = softcap * tanhf(s * inv_cap);
     const float mn = fmaxf(mx, s);
     const float corr = expf(mx - mn), p = expf(s - mn);
@@ -336,15 +459,15 @@ __global__ void softmax_attn_merge_kernel(const float* __restrict__ part_ml, con
 
 template <typename T, int R, int RV>
 static int sa_launch(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc,
-                     const int32_t* pos_ids, const float* sink, float scale, float softcap, int B, int Tn, int H, int G, int dim,
-                     int vdim, int window, int chunk, int ring, int splits, const DiffMaps& dm, float* scratch, void* y,
+                     const int32_t* pos_ids, const float* sink, const float* slopes, float scale, float softcap, int B, int Tn, int H,
+                     int G, int dim, int vdim, int window, int chunk, int ring, int splits, const DiffMaps& dm, float* scratch, void* y,
                      cudaStream_t st) {
   const int pairs = B * Tn * H * dm.maps;
   float* part_ml = scratch;
   float* part_acc = scratch ? scratch + (size_t)pairs * splits * 2 : nullptr;
   const dim3 grid((pairs + SA_WARPS - 1) / SA_WARPS, splits);
   softmax_attn_kernel<T, R, RV><<<grid, SA_WARPS * 32, 0, st>>>((const T*)q, q_stride, (const T*)gate, gate_stride, (const T*)kc,
-                                                               (const T*)vc, pos_ids, sink, scale, softcap, Tn, H, G, dim, vdim, window,
+                                                               (const T*)vc, pos_ids, sink, slopes, scale, softcap, Tn, H, G, dim, vdim, window,
                                                                chunk, ring, splits, dm.maps, pairs, part_ml, part_acc, (T*)y);
   LL_LAUNCH_OK("softmax_attn_kernel");
   if (splits > 1 || dm.maps > 1) {
@@ -358,13 +481,13 @@ static int sa_launch(const void* q, int q_stride, const void* gate, int gate_str
 
 template <typename T>
 static int sa_dispatch(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc,
-                       const int32_t* pos_ids, const float* sink, float scale, float softcap, int B, int Tn, int H, int G, int dim,
-                       int vdim, int window, int chunk, int ring, int splits, const DiffMaps& dm, float* scratch, void* y,
+                       const int32_t* pos_ids, const float* sink, const float* slopes, float scale, float softcap, int B, int Tn, int H,
+                       int G, int dim, int vdim, int window, int chunk, int ring, int splits, const DiffMaps& dm, float* scratch, void* y,
                        cudaStream_t st) {
   const int r = dim <= 64 ? 1 : dim <= 128 ? 2 : 4, rv = vdim <= 64 ? 1 : vdim <= 128 ? 2 : 4;
 #define LL_SA(RR, RRV)                                                                                                              \
   if (r == RR && rv == RRV)                                                                                                         \
-    return sa_launch<T, RR, RRV>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, scale, softcap, B, Tn, H, G, dim, vdim, window, \
+    return sa_launch<T, RR, RRV>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, slopes, scale, softcap, B, Tn, H, G, dim, vdim, window, \
                                  chunk, ring, splits, dm, scratch, y, st);
   LL_SA(1, 1) LL_SA(1, 2) LL_SA(1, 4) LL_SA(2, 1) LL_SA(2, 2) LL_SA(2, 4) LL_SA(4, 1) LL_SA(4, 2) LL_SA(4, 4)
 #undef LL_SA
@@ -409,12 +532,13 @@ __device__ __forceinline__ float tm_tanh(float x) { return 1.f - __fdividef(2.f,
 // MAPS = 2: the block walks its keys once per map (queries and keys of the map, the same values) and keeps the first map's
 // normalised output in registers until the second is there; the difference, its unit norm and `post` are the epilogue.
 // DK / DV: the padded sizes of a key row and of a value row (a map's keys may be half as wide as the values).
-template <int DK, int DV, int MAPS>
+// BIAS: scores carry the distance bias (an instantiation of its own: the plain one keeps its registers).
+template <int DK, int DV, int MAPS, bool BIAS>
 __global__ void __launch_bounds__(TM_THREADS, MAPS == 1 ? 3 : 2) softmax_attn_mma_kernel(
     const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ gate, int gate_stride,
     const __nv_bfloat16* __restrict__ kc, const __nv_bfloat16* __restrict__ vc, const int32_t* __restrict__ pos_ids,
-    const float* __restrict__ sink, float scale, float softcap, int Tn, int H, int G, int dim, int vdim, int window, int chunk, int ring,
-    float lambda, float post, float eps, __nv_bfloat16* __restrict__ y) {
+    const float* __restrict__ sink, const float* __restrict__ slopes, float scale, float softcap, int Tn, int H, int G, int dim, int vdim,
+    int window, int chunk, int ring, float lambda, float post, float eps, __nv_bfloat16* __restrict__ y) {
   constexpr int LD = DK + 8, CH = DK / 8, LV = DV + 8, CV = DV / 8, STAGE = TM_K * (LD + LV);      // a stage: 64 key rows, then 64 value rows
   extern __shared__ __align__(16) unsigned char tm_smem[];
   __nv_bfloat16* const stages = (__nv_bfloat16*)tm_smem;
@@ -430,6 +554,7 @@ __global__ void __launch_bounds__(TM_THREADS, MAPS == 1 ? 3 : 2) softmax_attn_mm
   const int wlo = sa_first_visible(p0 + warp * 16, window, chunk), whi = p0 + warp * 16 + 15;     // what the warp's rows can see
   const int khi = p0 + nq - 1;
   const float inv_cap = softcap > 0.f ? 1.f / softcap : 0.f;
+  const float slope = BIAS ? slopes[h] : 0.f;
   const int wlo_last = sa_first_visible(whi, window, chunk);
   const int kt0 = sa_first_visible(p0, window, chunk);
   const __nv_bfloat16* vbase = vc + ((size_t)b * ring * G + g) * vdim;
@@ -503,6 +628,8 @@ __global__ void __launch_bounds__(TM_THREADS, MAPS == 1 ? 3 : 2) softmax_attn_mm
         }
       }
       float tmax[2] = {-INFINITY, -INFINITY};
+      // key position minus query position of the fragment's first column (whole numbers: exact)
+      const float d0[2] = {(float)(kt + (lane & 3) * 2 - qp[0]), (float)(kt + (lane & 3) * 2 - qp[1])};
 #pragma unroll
       for (int n = 0; n < TM_K / 8; ++n)
 #pragma unroll
@@ -510,6 +637,7 @@ __global__ void __launch_bounds__(TM_THREADS, MAPS == 1 ? 3 : 2) softmax_attn_mm
           const int rr = e >> 1;
           const int kp = kt + n * 8 + (lane & 3) * 2 + (e & 1);
           float v = sc[n][e] * scale;
+          if (BIAS) v = fmaf(slope, d0[rr] + (float)(n * 8 + (e & 1)), v);
           if (softcap > 0.f) v = softcap * tm_tanh(v * inv_cap);
           if (!full) v = (kp <= qp[rr] && kp >= qlo[rr]) ? v : -INFINITY;
           sc[n][e] = v;
@@ -617,20 +745,21 @@ __global__ void __launch_bounds__(TM_THREADS, MAPS == 1 ? 3 : 2) softmax_attn_mm
   }  // maps
 }
 
-template <int DK, int DV, int MAPS>
+template <int DK, int DV, int MAPS, bool BIAS = false>
 static int tm_launch(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, const int32_t* pos_ids,
-                     const float* sink, float scale, float softcap, int B, int Tn, int H, int G, int dim, int vdim, int window, int chunk,
+                     const float* sink, const float* slopes, float scale, float softcap, int B, int Tn, int H, int G, int dim, int vdim,
+                     int window, int chunk,
                      int ring, const DiffMaps& dm, void* y, cudaStream_t st) {
   const dim3 grid((Tn + TM_Q - 1) / TM_Q, H, B);
   constexpr int smem = 2 * TM_K * (DK + 8 + DV + 8) * (int)sizeof(__nv_bfloat16);
   static bool sized = false;
   if (!sized) {
-    LL_CUDA(cudaFuncSetAttribute(softmax_attn_mma_kernel<DK, DV, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    LL_CUDA(cudaFuncSetAttribute(softmax_attn_mma_kernel<DK, DV, MAPS, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     sized = true;
   }
-  softmax_attn_mma_kernel<DK, DV, MAPS><<<grid, TM_THREADS, smem, st>>>(
+  softmax_attn_mma_kernel<DK, DV, MAPS, BIAS><<<grid, TM_THREADS, smem, st>>>(
       (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)gate, gate_stride, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc,
-      pos_ids, sink, scale, softcap, Tn, H, G, dim, vdim, window, chunk, ring, dm.lambda, dm.post, dm.eps, (__nv_bfloat16*)y);
+      pos_ids, sink, slopes, scale, softcap, Tn, H, G, dim, vdim, window, chunk, ring, dm.lambda, dm.post, dm.eps, (__nv_bfloat16*)y);
   LL_LAUNCH_OK("softmax_attn_mma_kernel");
   return LL_OK;
 }
@@ -684,6 +813,38 @@ int ll_qk_rotary_append(const void* q, int q_stride, const void* k, int k_stride
                                   vc, B, T, H, G, dim, vdim, ring, 1, stream);
 }
 
+int ll_qk_head_append(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const void* first,
+                      int first_stride, float lam, int dtype, const float* q_norm, const float* k_norm, float eps, const float* freq,
+                      int rot_dims, float temp_coef, int temp_every, const int32_t* pos_ids, void* q_out, void* kc, void* vc, int B, int T,
+                      int H, int G, int dim, int vdim, int ring, ll_stream stream) {
+  LL_CHECK_ARG(q && k && v && q_out && kc && vc && pos_ids && B >= 0 && T >= 0 && H > 0 && G > 0 && dim > 0 && vdim > 0 && ring > 0 &&
+                   temp_every >= 0,
+               "bad qk_head_append arguments");
+  LL_CHECK_ARG(rot_dims >= 0 && rot_dims <= dim && rot_dims % 2 == 0 && (rot_dims == 0 || freq), "qk_head_append: bad rotation");
+  if (dim > QH_DIM) {
+    set_error("qk_head_append: heads of %d dimensions (up to %d)", dim, QH_DIM);
+    return LL_ERR_UNSUPPORTED;
+  }
+  if (B == 0 || T == 0) return LL_OK;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int pair = ((q_stride | k_stride | v_stride | (first ? first_stride : 0) | dim | vdim) & 1) == 0 &&
+                   (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)first | (uintptr_t)q_out | (uintptr_t)kc | (uintptr_t)vc) & 3) == 0;
+#define LL_QH(T_)                                                                                                                     \
+  qk_head_append_kernel<T_><<<B * T, QP_THREADS, 0, st>>>((const T_*)q, q_stride, (const T_*)k, k_stride, (const T_*)v, v_stride,      \
+                                                          (const T_*)first, first_stride, lam, q_norm, k_norm, eps, freq, rot_dims,    \
+                                                          temp_coef, temp_every, pos_ids, (T_*)q_out, (T_*)kc, (T_*)vc, T, H, G, dim,  \
+                                                          vdim, ring, pair)
+  if (dtype == LL_F32) LL_QH(float);
+  else if (dtype == LL_BF16) LL_QH(__nv_bfloat16);
+  else {
+    set_error("qk_head_append: unsupported dtype %d", dtype);
+    return LL_ERR_UNSUPPORTED;
+  }
+#undef LL_QH
+  LL_LAUNCH_OK("qk_head_append_kernel");
+  return LL_OK;
+}
+
 int ll_softmax_attn_tensor_form(int dtype, int T, int dim, int vdim, int q_stride, int gate_stride, int splits) {
   return tm_supported(dtype, T, dim, vdim, q_stride, gate_stride, splits) ? 1 : 0;
 }
@@ -693,10 +854,10 @@ size_t ll_softmax_attn_scratch_bytes(int M, int H, int vdim, int splits) {
   return (size_t)M * H * splits * (2 + (size_t)vdim) * sizeof(float);
 }
 
-int ll_softmax_attn_maps(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, int dtype,
-                         const int32_t* pos_ids, const float* sink, float scale, float softcap, int B, int T, int H, int G, int dim,
-                         int vdim, int window, int chunk, int ring, int splits, int form, int maps, float diff_lambda, float diff_post,
-                         float eps, float* scratch, void* y, ll_stream stream) {
+int ll_softmax_attn_biased(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, int dtype,
+                           const int32_t* pos_ids, const float* sink, const float* slopes, float scale, float softcap, int B, int T, int H,
+                           int G, int dim, int vdim, int window, int chunk, int ring, int splits, int form, int maps, float diff_lambda,
+                           float diff_post, float eps, float* scratch, void* y, ll_stream stream) {
   LL_CHECK_ARG(q && kc && vc && pos_ids && y, "softmax_attn: null pointer");
   LL_CHECK_ARG(B >= 0 && T >= 0 && H > 0 && G > 0 && H % G == 0 && dim > 0 && vdim > 0 && ring > 0 && window >= 0 && chunk >= 0 &&
                    splits >= 1 && splits <= SA_MAX_SPLITS && (maps == 1 || maps == 2),
@@ -708,19 +869,21 @@ int ll_softmax_attn_maps(const void* q, int q_stride, const void* gate, int gate
   if (B == 0 || T == 0) return LL_OK;
   cudaStream_t st = (cudaStream_t)stream;
   const DiffMaps dm{maps, diff_lambda, diff_post, eps};
-  if (form == 0 && tm_supported(dtype, T, dim, vdim, q_stride, gate ? gate_stride : 0, splits)) {
+  if (form == 0 && !(slopes && maps > 1) && tm_supported(dtype, T, dim, vdim, q_stride, gate ? gate_stride : 0, splits)) {
     const int d = dim > vdim ? dim : vdim;
     if (maps == 1) {           // one map: key and value rows padded alike
-#define LL_TM(DD)                                                                                                                   \
-  if (d <= DD)                                                                                                                      \
-    return tm_launch<DD, DD, 1>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, scale, softcap, B, T, H, G, dim, vdim, window, \
-                                chunk, ring, dm, y, st);
+#define LL_TM_B(DD, BB)                                                                                                               \
+  tm_launch<DD, DD, 1, BB>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, slopes, scale, softcap, B, T, H, G, dim, vdim, window, \
+                           chunk, ring, dm, y, st)
+#define LL_TM(DD) \
+  if (d <= DD) return slopes ? LL_TM_B(DD, true) : LL_TM_B(DD, false);
       LL_TM(32) LL_TM(64) LL_TM(96) LL_TM(128)
 #undef LL_TM
+#undef LL_TM_B
     }
 #define LL_TM2(KK, VV)                                                                                                              \
   if (dim <= KK && vdim <= VV)                                                                                                      \
-    return tm_launch<KK, VV, 2>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, scale, softcap, B, T, H, G, dim, vdim, window, \
+    return tm_launch<KK, VV, 2>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, slopes, scale, softcap, B, T, H, G, dim, vdim, window, \
                                 chunk, ring, dm, y, st);
 #define LL_TM2_ROW(KK) LL_TM2(KK, 32) LL_TM2(KK, 64) LL_TM2(KK, 96) LL_TM2(KK, 128)
     LL_TM2_ROW(32) LL_TM2_ROW(64) LL_TM2_ROW(96) LL_TM2_ROW(128)
@@ -729,13 +892,21 @@ int ll_softmax_attn_maps(const void* q, int q_stride, const void* gate, int gate
   }
   LL_CHECK_ARG(scratch || (splits == 1 && maps == 1), "softmax_attn: split key ranges and several maps meet in scratch memory");
   if (dtype == LL_F32)
-    return sa_dispatch<float>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, scale, softcap, B, T, H, G, dim, vdim, window, chunk,
+    return sa_dispatch<float>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, slopes, scale, softcap, B, T, H, G, dim, vdim, window, chunk,
                               ring, splits, dm, scratch, y, st);
   if (dtype == LL_BF16)
-    return sa_dispatch<__nv_bfloat16>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, scale, softcap, B, T, H, G, dim, vdim, window,
+    return sa_dispatch<__nv_bfloat16>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, slopes, scale, softcap, B, T, H, G, dim, vdim, window,
                                       chunk, ring, splits, dm, scratch, y, st);
   set_error("softmax_attn: unsupported dtype %d", dtype);
   return LL_ERR_UNSUPPORTED;
+}
+
+int ll_softmax_attn_maps(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, int dtype,
+                         const int32_t* pos_ids, const float* sink, float scale, float softcap, int B, int T, int H, int G, int dim,
+                         int vdim, int window, int chunk, int ring, int splits, int form, int maps, float diff_lambda, float diff_post,
+                         float eps, float* scratch, void* y, ll_stream stream) {
+  return ll_softmax_attn_biased(q, q_stride, gate, gate_stride, kc, vc, dtype, pos_ids, sink, nullptr, scale, softcap, B, T, H, G, dim, vdim,
+                                window, chunk, ring, splits, form, maps, diff_lambda, diff_post, eps, scratch, y, stream);
 }
 
 int ll_softmax_attn(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, int dtype,

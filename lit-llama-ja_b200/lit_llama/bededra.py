@@ -316,7 +316,7 @@ class Bededra(PortionedDecoder):
             else:
                 u = h1
             if blk.kind == "mamba2":
-                pending = blk.mix(u, B, T, pos_ids, self.states[si:si + 2])
+                pending = [(blk.mix(u, B, T, pos_ids, self.states[si:si + 2]), 1.0)]
                 si += 2
             else:
                 spec = blk.mix.left.spec

@@ -13,6 +13,9 @@
       o_t = S_t^T q_t / (max(|n_t . q_t|, e^(-mx_t)) + 1e-6),  q_t = W_q h * dim^(-1/2)
       out = W_o ( headnorm(o) * w * sigmoid(W_g h) )
   The normaliser n rides in the same walk as one more value column that is constantly 1.
+* ``ConstantDecayAttention`` - linear attention with one constant decay per head ("lightning" form):
+      q, k, v = silu(W_q h), silu(W_k h), silu(W_v h);  S_t = decay_h S_(t-1) + k_t v_t^T;  o_t = S_t^T q_t
+      out = W_o ( rmsnorm(all heads together) * w * sigmoid(W_g h) )
 
 Decays, step sizes, the state, the read-out and the norms are fp32; the projections, the short convolution's output and
 the gates are in the activation dtype.  A sequence at position 0 starts from a zero state whatever its slot holds.
@@ -42,6 +45,16 @@ def decay_scan(q, q_col, k, k_col, v, v_col, decay, per_channel, kscale, skip, q
     N.call("ll_decay_scan", N.ptr_at(q, q_col), q.stride(0), N.ptr_at(k, k_col), k.stride(0), N.ptr_at(v, v_col), v.stride(0),
            N.dtype_code(v.dtype), N.ptr(decay), 1 if per_channel else 0, N.ptr(kscale), N.ptr(skip), float(qscale), N.ptr(state),
            N.ptr(pos_ids), N.ptr(y), B, T, H, qk_heads, n, p, 1 if unit_col else 0, N.stream())
+    return y
+
+
+def decay_scan_constant(proj, q_col, k_col, v_col, decay, silu, qscale, state, pos_ids, B, T, H, qk_heads, n, p):
+    """The same walk with one constant decay per head (``decay`` fp32 ``[H]``) over column slices of one projection output;
+    ``silu``: q, k and v pass it as they are read."""
+    y = torch.empty((B * T, H * p), dtype=torch.float32, device=proj.device)
+    N.call("ll_decay_scan_constant", N.ptr_at(proj, q_col), proj.stride(0), N.ptr_at(proj, k_col), proj.stride(0), N.ptr_at(proj, v_col),
+           proj.stride(0), N.dtype_code(proj.dtype), N.ptr(decay), 1 if silu else 0, float(qscale), N.ptr(state), N.ptr(pos_ids), N.ptr(y),
+           B, T, H, qk_heads, n, p, N.stream())
     return y
 
 
@@ -111,7 +124,7 @@ class StateSpaceMixer(nn.Module):
         self.norm.copy_(get("norm").float())
         self.w_o.copy_(get("o"))
 
-    def forward(self, u: torch.Tensor, B: int, T: int, pos_ids: torch.Tensor, states) -> List[Tuple[torch.Tensor, float]]:
+    def forward(self, u: torch.Tensor, B: int, T: int, pos_ids: torch.Tensor, states) -> torch.Tensor:
         s = self.spec
         conv_state, ssm_state = states
         M = B * T
@@ -125,7 +138,7 @@ class StateSpaceMixer(nn.Module):
         y = decay_scan(xbc, s.inner + gn, xbc, s.inner, xbc, 0, decay, False, dt, self.skip, 1.0, ssm_state, pos_ids, B, T,
                        s.heads, s.groups, s.state, s.vdim)
         out = gated_group_norm(y, proj, 0, self.norm, False, s.eps, s.norm_groups, True, u.dtype)
-        return [(F.linear(out, self.w_o), 1.0)]
+        return F.linear(out, self.w_o)
 
 
 @dataclass
@@ -238,4 +251,54 @@ class MatrixMemoryMixer(nn.Module):
         y = decay_scan(proj, c["q"], proj, c["k"], proj, c["v"], keep, False, take, None, s.dim ** -0.5, memory, pos_ids, B, T,
                        s.heads, s.heads, s.dim, s.vdim + 1, unit_col=True)
         out = gated_group_norm(y, proj, c["g"], self.norm, False, s.eps, s.heads, False, proj.dtype, sigmoid=True, part=s.vdim, stab=stab)
+        return F.linear(out, self.w_o)
+
+
+@dataclass
+class ConstantDecaySpec:
+    width: int
+    heads: int
+    dim: int                # query / key channels per head
+    vdim: int
+    decay: Tuple[float, ...]
+    eps: float
+
+    def __post_init__(self):
+        self.decay = tuple(float(d) for d in self.decay)
+        if len(self.decay) != self.heads:
+            raise ValueError(f"{len(self.decay)} decays for {self.heads} heads")
+
+
+class ConstantDecayAttention(nn.Module):
+    def __init__(self, spec: ConstantDecaySpec, dtype: torch.dtype, device) -> None:
+        super().__init__()
+        s = self.spec = spec
+        kw = dict(dtype=dtype, device=device)
+        f32 = dict(dtype=torch.float32, device=device)
+        hd, hv = s.heads * s.dim, s.heads * s.vdim
+        self.cols = dict(q=0, k=hd, v=2 * hd, g=2 * hd + hv)
+        self.n_in = 2 * hd + 2 * hv
+        self.w_in = nn.Parameter(torch.zeros((pad8(self.n_in), s.width), **kw), requires_grad=False)
+        self.register_buffer("decay", torch.tensor(s.decay, dtype=torch.float64).to(**f32), persistent=False)
+        self.norm = nn.Parameter(torch.ones(hv, **f32), requires_grad=False)
+        self.w_o = nn.Parameter(torch.zeros((s.width, hv), **kw), requires_grad=False)
+
+    def state_shapes(self, B: int) -> List[Tuple[int, ...]]:
+        s = self.spec
+        return [(B, s.heads, s.dim, s.vdim)]
+
+    def load(self, get) -> None:
+        """``get(suffix)`` returns the tensor '<layer>.mix.<suffix>'."""
+        self.w_in.zero_()
+        self.w_in[: self.n_in].copy_(torch.cat([get(n).to(self.w_in.dtype) for n in self.cols], dim=0))
+        self.norm.copy_(get("norm").float())
+        self.w_o.copy_(get("o"))
+
+    def forward(self, u: torch.Tensor, B: int, T: int, pos_ids: torch.Tensor, states) -> torch.Tensor:
+        s = self.spec
+        c = self.cols
+        proj = F.linear(u, self.w_in)
+        y = decay_scan_constant(proj, c["q"], c["k"], c["v"], self.decay, True, 1.0, states[0], pos_ids, B, T, s.heads, s.heads, s.dim,
+                                s.vdim)
+        out = gated_group_norm(y, proj, c["g"], self.norm, False, s.eps, 1, False, proj.dtype, sigmoid=True)
         return F.linear(out, self.w_o)

@@ -43,6 +43,10 @@ def _builtin() -> None:
         from .bumulix import ARCHITECTURE, Bumulix
 
         register_architecture(ARCHITECTURE, Bumulix.from_dir)
+    if "Livasun" not in _FROM_DIR:
+        from .livasun import ARCHITECTURE, Livasun
+
+        register_architecture(ARCHITECTURE, Livasun.from_dir)
 
 
 def load_model_dir(path, dtype: torch.dtype = torch.bfloat16, device="cuda"):

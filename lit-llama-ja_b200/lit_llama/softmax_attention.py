@@ -2,10 +2,13 @@
 sigmoid gate on the heads' outputs, with the variations models differ in as parameters of the spec:
 
     q, k <- [shortconv]( W h )                       a short causal filter per channel, its last inputs kept as state
-    q, k <- rmsnorm_row(.) * w                       one norm over the WHOLE projection, before the heads are split
+    q, k <- rmsnorm_row(.) * w                       one norm over the WHOLE projection, before the heads are split, or
+    q, k <- rmsnorm_head(.) * w                      one per head, with a weight of the head's size shared by all heads
+    q    <- q * (1 + coef ln(floor((p + 1) / every) + 1))      at position p (query temperature)
     q, k <- rotate(., position)                      rotary.RotarySpec (partial dimensions, rescaled frequencies)
-    v     = W_v h,  or the keys as they are before the rotation (``own_values`` False)
-    s_h(i, j) = scale * q_h(i).k_g(j)  [-> cap * tanh(s / cap)]
+    v     = W_v h,  or the keys as they are before the rotation (``own_values`` False),  or, mixed with the values an
+            earlier layer projected for the same token, (1 - lam) * W_v h + lam * v_first (lam learned; the mix is cached)
+    s_h(i, j) = scale * q_h(i).k_g(j)  [- slope_h * (i - j)]  [-> cap * tanh(s / cap)],     slope_h = 2^(-8 (h + 1) / H)
     visible:    j <= i  [and i - j < window]  [and j // chunk == i // chunk]
     w = exp(s) / (sum_visible exp(s) [+ exp(sink_h)])         the sink is a learned number per head without key or value
     out = W_o( concat_h( sum_j w v_g(j) ) * sigmoid(W_g h) )
@@ -61,6 +64,11 @@ class SoftmaxAttentionSpec:
     maps: int = 1                        # score maps per head; 2: the difference of two softmax maps with a unit norm per head
     diff: float = 0.0                    # the constant of the two-map combination
     gate: bool = True                    # sigmoid(W_g h) on the heads' outputs
+    head_norm: bool = False              # a norm per head on q and k (qk_norm: over the whole projection)
+    temp_coef: float = 0.0               # query temperature
+    temp_every: int = 0                  # 0: none
+    distance_bias: bool = False          # scores fall by slope_h per position of distance
+    v_mix: bool = False                  # values are mixed with those of another layer (``attend``'s ``first_values``)
 
     def __post_init__(self):
         if self.heads % self.kv_heads:
@@ -71,8 +79,19 @@ class SoftmaxAttentionSpec:
             raise ValueError(f"{self.maps} score maps per head (1 or 2)")
         if self.maps > 1 and not self.own_values:
             raise ValueError("values taken from the keys need one score map per head")
+        per_head = self.head_norm or self.temp_every > 0 or self.v_mix
+        if per_head and (self.qk_norm or self.maps > 1 or not self.own_values or self.kv_from is not None):
+            raise ValueError("a norm per head, a query temperature and mixed values go with one score map, keys and values of the "
+                             "layer's own and no norm over the whole projection")
+        if self.temp_every < 0:
+            raise ValueError(f"a query temperature that steps every {self.temp_every} positions")
         if self.rotary.dims > self.dim:
             raise ValueError(f"{self.rotary.dims} rotated dimensions in heads of {self.dim}")
+
+    @property
+    def by_head(self) -> bool:
+        """Whether q, k and v are prepared head by head (ll_qk_head_append)."""
+        return self.head_norm or self.temp_every > 0 or self.v_mix
 
     @property
     def reach(self) -> Optional[int]:
@@ -99,13 +118,17 @@ class SoftmaxAttention(nn.Module):
         self.w_in = nn.Parameter(torch.zeros((pad8(self.n_in), s.width), **kw), requires_grad=False)
         self.conv_channels = hd + (gd if self.owner else 0)
         self.conv = ShortConv(self.conv_channels, s.conv_taps, False, device) if s.conv_taps > 0 else None
-        self.q_norm = nn.Parameter(torch.ones(hd, **f32), requires_grad=False) if s.qk_norm else None
-        self.k_norm = nn.Parameter(torch.ones(gd, **f32), requires_grad=False) if s.qk_norm and self.owner else None
+        normed = s.qk_norm or s.head_norm
+        self.q_norm = nn.Parameter(torch.ones(s.dim if s.head_norm else hd, **f32), requires_grad=False) if normed else None
+        self.k_norm = nn.Parameter(torch.ones(s.dim if s.head_norm else gd, **f32), requires_grad=False) if normed and self.owner else None
+        self.v_lambda = 0.0                            # lam of the value mix, read at load time
+        self.register_buffer("slopes", torch.tensor([2.0 ** (-8.0 * (h + 1) / s.heads) for h in range(s.heads)],
+                                                    dtype=torch.float64).to(**f32) if s.distance_bias else None, persistent=False)
         self.sink = nn.Parameter(torch.zeros(s.heads * s.maps, **f32), requires_grad=False) if s.sink else None
         self.register_buffer("freq", s.rotary.frequencies(device), persistent=False)
         self.diff_lambda = 0.0                         # lam of the two-map combination, formed at load time
         # queries that are neither filtered, normed nor turned are read where the input projection left them
-        self.plain_q = self.conv is None and not s.qk_norm and s.rotary.dims == 0
+        self.plain_q = self.conv is None and not s.qk_norm and s.rotary.dims == 0 and not s.by_head
         self.w_o = nn.Parameter(torch.zeros((s.width, hv), **kw), requires_grad=False)
 
     def state_shapes(self, B: int) -> List[Tuple[int, ...]]:
@@ -131,15 +154,23 @@ class SoftmaxAttention(nn.Module):
         if s.maps == 2:
             l = [get(n).double() for n in ("lq1", "lk1", "lq2", "lk2")]
             self.diff_lambda = float(torch.exp((l[0] * l[1]).sum()) - torch.exp((l[2] * l[3]).sum()) + s.diff)
+        if s.v_mix:
+            self.v_lambda = float(get("vmix").float())
         self.w_o.copy_(get("o"))
+
+    def values(self, proj: torch.Tensor) -> torch.Tensor:
+        """The columns of the input projection's output that hold this layer's own values."""
+        s = self.spec
+        return proj[:, self.cols["v"]: self.cols["v"] + s.kv_heads * s.vdim]
 
     def forward(self, u: torch.Tensor, B: int, T: int, pos_ids: torch.Tensor, caches, conv_state=None, splits: int = 1,
                 form: int = 0) -> torch.Tensor:
         return F.linear(self.attend(F.linear(u, self.w_in), B, T, pos_ids, caches, conv_state, splits, form), self.w_o)
 
     def attend(self, proj: torch.Tensor, B: int, T: int, pos_ids: torch.Tensor, caches, conv_state=None, splits: int = 1,
-               form: int = 0) -> torch.Tensor:
-        """``proj``: the stacked input projection's output; ``caches`` = (keys, values) of this layer or of the one it reads.
+               form: int = 0, first_values: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``proj``: the stacked input projection's output; ``caches`` = (keys, values) of this layer or of the one it reads;
+        ``first_values``: the values mixed into this layer's (``v_mix``), of the same tokens.
         Returns the gated heads ``[B*T, heads * vdim]`` (before the output projection)."""
         s = self.spec
         c = self.cols
@@ -161,10 +192,20 @@ class SoftmaxAttention(nn.Module):
         else:
             q = torch.empty((M, hd), dtype=proj.dtype, device=proj.device)
             q_ptr, q_stride = N.ptr(q), hd
-        if self.owner or not self.plain_q:
+        if s.by_head:
+            if s.v_mix and (first_values is None or first_values.shape != (M, s.kv_heads * s.vdim)):
+                raise ValueError("a layer with mixed values needs the other layer's values of the same tokens")
+            first = first_values if s.v_mix else None
+            N.call("ll_qk_head_append", q_at, src.stride(0), k_at, src.stride(0), v_at, proj.stride(0), N.ptr(first),
+                   first.stride(0) if first is not None else 0, float(self.v_lambda), dtc,
+                   N.ptr(self.q_norm), N.ptr(self.k_norm), float(s.eps), N.ptr(self.freq), s.rotary.dims, float(s.temp_coef),
+                   s.temp_every, N.ptr(pos_ids), N.ptr(q), N.ptr(kc), N.ptr(vc), B, T, s.heads, s.kv_heads, s.dim, s.vdim, ring, st)
+        elif self.owner or not self.plain_q:
             N.call("ll_qk_rotary_append_maps", None if self.plain_q else q_at, src.stride(0), k_at if self.owner else None, src.stride(0),
                    v_at, proj.stride(0), dtc, N.ptr(self.q_norm), N.ptr(self.k_norm), float(s.eps), N.ptr(self.freq), s.rotary.dims,
                    N.ptr(pos_ids), N.ptr(q), N.ptr(kc), N.ptr(vc), B, T, s.heads, s.kv_heads, s.dim, s.vdim, ring, s.maps, st)
+        if s.distance_bias and s.maps > 1:
+            form = 1                                   # two biased maps have no tensor-core form
         gate_at, gate_stride = (N.ptr_at(proj, c["g"]), proj.stride(0)) if s.gate else (None, 0)
         scratch = None
         if splits > 1 or (s.maps > 1 and (form != 0 or not N.call_ret("ll_softmax_attn_tensor_form", dtc, T, s.dim, s.vdim, q_stride,
@@ -172,7 +213,7 @@ class SoftmaxAttention(nn.Module):
             scratch = torch.empty(N.call_ret("ll_softmax_attn_scratch_bytes", M, s.heads * s.maps, s.vdim, splits) // 4,
                                   dtype=torch.float32, device=proj.device)
         y = torch.empty((M, s.heads * s.vdim), dtype=proj.dtype, device=proj.device)
-        N.call("ll_softmax_attn_maps", q_ptr, q_stride, gate_at, gate_stride, N.ptr(kc), N.ptr(vc), dtc, N.ptr(pos_ids),
-               N.ptr(self.sink), float(s.scale), float(s.softcap), B, T, s.heads, s.kv_heads, s.dim, s.vdim, s.window or 0, s.chunk or 0,
-               ring, splits, form, s.maps, float(self.diff_lambda), float(1.0 - s.diff), float(s.eps), N.ptr(scratch), N.ptr(y), st)
+        N.call("ll_softmax_attn_biased", q_ptr, q_stride, gate_at, gate_stride, N.ptr(kc), N.ptr(vc), dtc, N.ptr(pos_ids),
+               N.ptr(self.sink), N.ptr(self.slopes), float(s.scale), float(s.softcap), B, T, s.heads, s.kv_heads, s.dim, s.vdim,
+               s.window or 0, s.chunk or 0, ring, splits, form, s.maps, float(self.diff_lambda), float(1.0 - s.diff), float(s.eps), N.ptr(scratch), N.ptr(y), st)
         return y

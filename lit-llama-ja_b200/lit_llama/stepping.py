@@ -11,12 +11,13 @@ from __future__ import annotations
 import contextlib
 import gc
 import os
-from typing import Dict, Optional
+from typing import Dict, List, Optional, Tuple
 
 import torch
 import torch.nn as nn
 
 from . import _native as N
+from .cache import TensorPool, max_portion, ring_length
 
 
 @contextlib.contextmanager
@@ -143,6 +144,80 @@ class PortionedDecoder(nn.Module):
             self._forward_portion(s_idx, s_pos, None)
 
 
+class RingStateDecoder(PortionedDecoder):
+    """A model whose per-sequence memory is fp32 recurrent state (``states``: every layer's tensors in order) and key / value
+    rings in the activation dtype (``kv_caches``: (keys, values) of every ring in order), each as long as the furthest look-back
+    among its readers and a pass of ``prefill_portion`` tokens ask for.  All of it comes from the package's ``TensorPool`` with
+    stable addresses and is written in place; nothing is cleared between requests: the kernels start a sequence from nothing
+    when its first position is 0.  A model sets ``config``, ``dtype``, ``device`` and says what its memory looks like."""
+
+    def __init__(self) -> None:
+        super().__init__()
+        self._pool = TensorPool(max_sets=4, on_evict=self._drop_graphs)
+        self.states: List[torch.Tensor] = []
+        self.kv_caches: List[torch.Tensor] = []
+        self._rings: Tuple[int, ...] = ()
+        self._batch = 0
+
+    # ------------------------------------------------------------------ hooks
+    def _ring_reaches(self) -> List[Optional[int]]:
+        """Per ring: no reader's query at position i sees a key before ``i - reach + 1`` (None: unbounded)."""
+        raise NotImplementedError
+
+    def _ring_shapes(self, n: int, B: int, ring: int) -> List[Tuple[int, ...]]:
+        """(keys, values) of ring ``n`` with ``ring`` slots."""
+        raise NotImplementedError
+
+    def _state_shapes(self, B: int) -> List[Tuple[int, ...]]:
+        raise NotImplementedError
+
+    # ------------------------------------------------------------------ memory
+    def reset_cache(self) -> None:
+        """The sequences end: their slots are given back (the tensors stay allocated; the next sequence starts at position
+        0, where the kernels take nothing from them)."""
+        self.states, self.kv_caches, self._rings, self._batch = [], [], (), 0
+
+    def _ring_plan(self, max_seq_length: int) -> Tuple[int, ...]:
+        portion = min(self.prefill_portion, max_seq_length)
+        return tuple(max(1, ring_length(max_seq_length, r, portion)) for r in self._ring_reaches())
+
+    def _begin(self, B: int, max_seq_length: int, keep: bool) -> None:
+        rings = self._ring_plan(max_seq_length)
+        if (self.states or self.kv_caches) and self._batch == B and self._rings == rings:
+            return
+        st_shapes = self._state_shapes(B)
+        kv_shapes = [s for n, ring in enumerate(rings) for s in self._ring_shapes(n, B, ring)]
+        if keep:
+            self.states = self._pool.get(st_shapes, torch.float32, self.device, zero=False) if st_shapes else []
+            self.kv_caches = self._pool.get(kv_shapes, self.dtype, self.device, zero=False) if kv_shapes else []
+        else:                      # a forward that keeps nothing: scratch memory, the pool's sets stay as they are
+            self.states = [torch.empty(s, dtype=torch.float32, device=self.device) for s in st_shapes]
+            self.kv_caches = [torch.empty(s, dtype=self.dtype, device=self.device) for s in kv_shapes]
+        self._rings, self._batch = rings, B
+
+    def _piece(self, max_seq_length: int) -> int:
+        return min([max_seq_length] + [max_portion(ring, max_seq_length, r) for r, ring in zip(self._ring_reaches(), self._rings)])
+
+    def _graph_key(self, B: int) -> tuple:
+        return (B, self._rings, self.states[0].data_ptr() if self.states else 0, self.kv_caches[0].data_ptr() if self.kv_caches else 0)
+
+    def _save_memory(self):
+        saved = (self.states, self.kv_caches, self._rings, self._batch)
+        self.states, self.kv_caches, self._rings, self._batch = [], [], (), 0
+        return saved
+
+    def _restore_memory(self, saved) -> None:
+        self.states, self.kv_caches, self._rings, self._batch = saved
+
+    def _warm_step(self, s_idx, s_pos) -> None:
+        """The eager runs before a capture advance the recurrent state; put it back afterwards (the ring row they write is
+        the one the real step writes again)."""
+        kept = [t.clone() for t in self.states]
+        super()._warm_step(s_idx, s_pos)
+        for t, k in zip(self.states, kept):
+            t.copy_(k)
+
+
 def head_logits(xn: torch.Tensor, head: torch.Tensor, vocab: int) -> torch.Tensor:
     """fp32 logits ``[rows, vocab]`` of normed rows ``xn`` against ``head`` (``[vocab rounded up to 8, width]``, zero rows
     at the end: the library's fast GEMMs want aligned outputs)."""
@@ -163,6 +238,13 @@ def add_norm_pair(x, branches, w1, w2, eps, out1, out2, act_dtype) -> None:
     b = list(branches) + [(None, 0.0)] * (3 - len(branches))
     N.call("ll_add_norm_pair", N.ptr(x), N.ptr(b[0][0]), float(b[0][1]), N.ptr(b[1][0]), float(b[1][1]), N.ptr(b[2][0]), float(b[2][1]),
            N.ptr(w1), N.ptr(w2), float(eps), N.ptr(out1), 1 if (out1 is not None and out1.dtype == torch.float32) else 0, N.ptr(out2),
+           N.dtype_code(act_dtype), x.shape[0], x.shape[1], N.stream())
+
+
+def add_layer_norm(x, branch, scale, w, b, eps, out, act_dtype) -> None:
+    """``x += scale * branch`` in place (fp32; ``branch`` None: nothing is added); then, with ``out`` given, ``out`` = the layer
+    norm of ``x`` with weight ``w`` and bias ``b``."""
+    N.call("ll_add_layer_norm", N.ptr(x), N.ptr(branch), float(scale), N.ptr(w), N.ptr(b), float(eps), N.ptr(out),
            N.dtype_code(act_dtype), x.shape[0], x.shape[1], N.stream())
 
 

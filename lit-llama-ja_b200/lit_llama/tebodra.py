@@ -14,9 +14,8 @@ Feed-forward: ``W_down gelu(W_up h)`` (erf form).  Output: ``head . (rmsnorm(x) 
 stored around zero; ``1 + w`` is formed once at load time in fp32.
 
 Per-sequence memory: key / value rings of the attention layers that own them (a borrowing layer holds none), the inputs of
-the short filters, the matrix memories with their normalisers and stabilisers.  All of it lives in tensors from the package's
-``TensorPool`` with stable addresses, written in place; nothing is cleared between requests: the kernels start a sequence
-from nothing when its first position is 0.  ``forward`` is the package's common step function (stepping.PortionedDecoder).
+the short filters, the matrix memories with their normalisers and stabilisers (stepping.RingStateDecoder, whose step function
+is the package's common one).
 """
 from __future__ import annotations
 
@@ -29,12 +28,11 @@ import torch
 import torch.nn as nn
 
 from . import _native as N
-from .cache import TensorPool, max_portion, ring_length
 from .feed_forward import DenseFF
 from .recurrence import MatrixMemoryMixer, MatrixMemorySpec, pad8
 from .rotary import RotarySpec
 from .softmax_attention import SoftmaxAttention, SoftmaxAttentionSpec
-from .stepping import PortionedDecoder, add_norm_pair, head_logits
+from .stepping import RingStateDecoder, add_norm_pair, head_logits
 
 ARCHITECTURE = "Tebodra"
 
@@ -151,7 +149,7 @@ class TebodraBlock(nn.Module):
             self.mlp.load(lambda s: get(p + "mlp." + s))
 
 
-class Tebodra(PortionedDecoder):
+class Tebodra(RingStateDecoder):
     architecture = ARCHITECTURE
 
     def __init__(self, config: TebodraConfig, dtype: torch.dtype = torch.bfloat16, device="cuda") -> None:
@@ -165,7 +163,6 @@ class Tebodra(PortionedDecoder):
         self.blocks = nn.ModuleList(TebodraBlock(i, l, config, dtype, self.device) for i, l in enumerate(config.layers))
         self.final_norm = nn.Parameter(torch.ones(config.width, dtype=torch.float32, device=self.device), requires_grad=False)
         self.head = nn.Parameter(torch.zeros((pad8(config.vocab), config.width), **kw), requires_grad=False)
-        self._pool = TensorPool(max_sets=4, on_evict=self._drop_graphs)
         # rings: one per attention layer with keys of its own, long enough for the furthest look-back among its readers
         self._owners = [i for i, l in enumerate(config.layers) if l.kind != "mlstm" and l.mixer.kv_from is None]
         self._reach: List[Optional[int]] = []
@@ -179,10 +176,6 @@ class Tebodra(PortionedDecoder):
         for i, l in enumerate(config.layers):
             if l.kind != "mlstm" and l.mixer.kv_from is not None:
                 self._cache_of[i] = self._cache_of[l.mixer.kv_from]
-        self.states: List[torch.Tensor] = []          # fp32, every layer's in order (filter inputs; memory, stabiliser)
-        self.kv_caches: List[torch.Tensor] = []       # (keys, values) of every owner in order
-        self._rings: Tuple[int, ...] = ()
-        self._batch = 0
 
     # ------------------------------------------------------------------ weights
     @torch.no_grad()
@@ -209,53 +202,14 @@ class Tebodra(PortionedDecoder):
         return model.eval()
 
     # ------------------------------------------------------------------ memory
-    def reset_cache(self) -> None:
-        """The sequences end: their slots are given back (the tensors stay allocated; the next sequence starts at position
-        0, where the kernels take nothing from them)."""
-        self.states, self.kv_caches, self._rings, self._batch = [], [], (), 0
+    def _ring_reaches(self) -> List[Optional[int]]:
+        return self._reach
 
-    def _ring_plan(self, max_seq_length: int) -> Tuple[int, ...]:
-        portion = min(self.prefill_portion, max_seq_length)
-        return tuple(max(1, ring_length(max_seq_length, r, portion)) for r in self._reach)
+    def _ring_shapes(self, n: int, B: int, ring: int) -> List[Tuple[int, ...]]:
+        return self.blocks[self._owners[n]].mix.cache_shapes(B, ring)
 
     def _state_shapes(self, B: int) -> List[Tuple[int, ...]]:
         return [s for b in self.blocks for s in b.mix.state_shapes(B)]
-
-    def _begin(self, B: int, max_seq_length: int, keep: bool) -> None:
-        rings = self._ring_plan(max_seq_length)
-        if (self.states or self.kv_caches) and self._batch == B and self._rings == rings:
-            return
-        st_shapes = self._state_shapes(B)
-        kv_shapes = [s for n, i in enumerate(self._owners) for s in self.blocks[i].mix.cache_shapes(B, rings[n])]
-        if keep:
-            self.states = self._pool.get(st_shapes, torch.float32, self.device, zero=False) if st_shapes else []
-            self.kv_caches = self._pool.get(kv_shapes, self.dtype, self.device, zero=False) if kv_shapes else []
-        else:                      # a forward that keeps nothing: scratch memory, the pool's sets stay as they are
-            self.states = [torch.empty(s, dtype=torch.float32, device=self.device) for s in st_shapes]
-            self.kv_caches = [torch.empty(s, dtype=self.dtype, device=self.device) for s in kv_shapes]
-        self._rings, self._batch = rings, B
-
-    def _piece(self, max_seq_length: int) -> int:
-        return min([max_seq_length] + [max_portion(ring, max_seq_length, r) for r, ring in zip(self._reach, self._rings)])
-
-    def _graph_key(self, B: int) -> tuple:
-        return (B, self._rings, self.states[0].data_ptr() if self.states else 0, self.kv_caches[0].data_ptr() if self.kv_caches else 0)
-
-    def _save_memory(self):
-        saved = (self.states, self.kv_caches, self._rings, self._batch)
-        self.states, self.kv_caches, self._rings, self._batch = [], [], (), 0
-        return saved
-
-    def _restore_memory(self, saved) -> None:
-        self.states, self.kv_caches, self._rings, self._batch = saved
-
-    def _warm_step(self, s_idx, s_pos) -> None:
-        """The eager runs before a capture advance the recurrent state; put it back afterwards (the ring row they write is
-        the one the real step writes again)."""
-        kept = [t.clone() for t in self.states]
-        super()._warm_step(s_idx, s_pos)
-        for t, k in zip(self.states, kept):
-            t.copy_(k)
 
     # ------------------------------------------------------------------ forward
     def _forward_portion(self, idx: torch.Tensor, pos_ids: torch.Tensor, sel) -> torch.Tensor:

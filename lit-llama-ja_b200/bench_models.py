@@ -1,6 +1,7 @@
 """Throughput of a model family beside its closest relative at equal size: prefill tokens/s, batch-1 decode tokens/s, and
 the hot kernels of each timed alone against the measured roofline.  ``bench.py --family lepalorn``: Lepalorn beside LLaMA;
-``bench.py --family bededra``: Bededra beside Lepalorn; ``bench.py --family tebodra``: Tebodra beside Bededra.  Random weights, layer shapes of real
+``bench.py --family bededra``: Bededra beside Lepalorn; ``bench.py --family tebodra``: Tebodra beside Bededra; ``--family bumulix``: Bumulix beside Tebodra; ``--family livasun``: Livasun
+beside Bededra.  Random weights, layer shapes of real
 models, a few layers each (every layer costs the same).  Timing: CUDA events, warm-up, an L2 flush (a 256 MB write)
 between timed iterations."""
 from __future__ import annotations
@@ -249,6 +250,48 @@ def bededra_model(s, device, dtype=torch.bfloat16):
     return m.eval()
 
 
+def moe_rows(moe, x, timer, add, tag):
+    """Router and both grouped GEMMs of one mixture layer, on the path the module takes for a step of this size."""
+    from lit_llama import _native as N
+
+    sp = moe.spec
+    T, E = x.shape
+    n = T * sp.top
+    add(f"moe router + sort {tag}", timer(lambda: moe.route(x), graph=True), 2.0 * T * sp.experts * E,
+        2.0 * T * E + 4.0 * sp.experts * E + 16.0 * n)
+    _, _, offsets, perm = moe.route(x)
+    h = torch.empty((n, sp.ff), dtype=x.dtype, device=x.device)
+    y = torch.empty((n, E), dtype=x.dtype, device=x.device)
+    tc = moe.takes_tensor_cores(n, x)
+    xs = torch.empty((n, E), dtype=x.dtype, device=x.device) if tc else None
+    up = moe.w_gu.shape[1]
+
+    def experts():
+        st = N.stream()
+        if tc:
+            N.call("ll_moe_gather_rows", N.ptr(x), E, N.ptr(perm), sp.top, n, E, N.ptr(xs), st)
+            N.call("ll_moe_grouped_gemm_tc", N.ptr(xs), N.ptr(moe.w_gu), N.ptr(offsets), N.ptr(perm), moe.up_mode, n, sp.experts, sp.ff, E,
+                   float(sp.limit), float(sp.alpha), N.ptr(h), sp.ff, st)
+            N.call("ll_moe_grouped_gemm_tc", N.ptr(h), N.ptr(moe.w_down), N.ptr(offsets), N.ptr(perm), 0, n, sp.experts, E, sp.ff, 0.0, 0.0,
+                   N.ptr(y), E, st)
+            return
+        N.call("ll_moe_grouped_gemm", N.ptr(x), E, N.ptr(moe.w_gu), N.ptr(offsets), N.ptr(perm), moe.up_mode, N.LL_BF16, n, sp.top,
+               sp.experts, sp.ff, E, float(sp.limit), float(sp.alpha), N.ptr(h), sp.ff, st)
+        N.call("ll_moe_grouped_gemm", N.ptr(h), sp.ff, N.ptr(moe.w_down), N.ptr(offsets), N.ptr(perm), 0, N.LL_BF16, n, sp.top, sp.experts,
+               E, sp.ff, 0.0, 0.0, N.ptr(y), E, st)
+
+    add(f"moe grouped GEMMs {tag}" + (" (tcgen05, with the row gather)" if tc else ""), timer(experts, graph=True),
+        2.0 * n * (up + sp.ff) * E, 2.0 * min(sp.experts, n) * (up + sp.ff) * E + 2.0 * n * (2 * E + 2 * sp.ff))
+
+
+def gated_norm_row(name, y, gate, gate_col, w, shared, groups, gate_first, sigmoid, timer, add):
+    from lit_llama.recurrence import gated_group_norm
+
+    T, C = y.shape
+    add(name, timer(lambda: gated_group_norm(y, gate, gate_col, w, shared, 1e-5, groups, gate_first, gate.dtype, sigmoid=sigmoid), graph=True),
+        0.0, 8.0 * T * C)
+
+
 def bededra_kernel_table(s, model, device, timer, prompt_len):
     """The mixers' kernels of one parallel and one mamba2 layer alone.  Roofline time = max(flops / tensor peak, bytes /
     copy bandwidth), flops and bytes counted for the mechanism (one sweep over the visible keys; one update and one
@@ -330,6 +373,12 @@ def bededra_kernel_table(s, model, device, timer, prompt_len):
                                            graph=True), 0.0, T * E * (4 + 4 + 2 + 2 + 4 + 2))
         cst = model.states[0]
         add(f"short_conv {tag}", timer(lambda: par.canon(h1, 0, cst, pos_ids, 1, T, bf, residual=True), graph=True), 0.0, T * E * (4 + 2))
+        pm = F.linear(x, mam.mix.w_in)
+        gated_norm_row(f"gated norm {tag} (state space)", torch.randn((T, ms.inner), device=device), pm, 0, mam.mix.norm, False, ms.norm_groups,
+                       True, False, timer, add)
+        gated_norm_row(f"gated norm {tag} (linear attention)", torch.randn((T, rs.heads * rs.vdim), device=device), proj, c0 + r.cols["g"],
+                       r.norm, True, rs.heads, False, False, timer, add)
+        moe_rows(par.mlp, x, timer, add, tag)
     return rows, which
 
 
@@ -695,8 +744,168 @@ def run_bumulix(args):
     return 0
 
 
+# Livasun at the widths of SIZES, four layers each: attention, state space, constant-decay linear attention, attention.
+# Attention heads and window as Bededra's, the state space too; linear attention with heads of 128 x 128 over the width.  The first
+# three layers carry experts (squared relu, as many and as large as Bededra's, with an always-on expert of half the chosen
+# experts' size: equal work per token), the last a silu-gated dense layer of the same work.
+LIVASUN_SIZES = {
+    "w1024": dict(width=1024, layers=4, heads=8, kv=2, dim=64, window=512, l_heads=8, l_dim=128, m_heads=32, m_vdim=64, state=128,
+                  experts=16, top=2, ff=768, groups=4, keep_groups=2),
+    "w2048": dict(width=2048, layers=4, heads=16, kv=4, dim=128, window=1024, l_heads=16, l_dim=128, m_heads=64, m_vdim=64, state=128,
+                  experts=32, top=4, ff=1024, groups=8, keep_groups=4),
+    "w4096": dict(width=4096, layers=4, heads=32, kv=8, dim=128, window=2048, l_heads=32, l_dim=128, m_heads=128, m_vdim=64, state=128,
+                  experts=32, top=4, ff=2048, groups=8, keep_groups=4),
+}
+
+
+def livasun_model(s, device, dtype=torch.bfloat16):
+    from lit_llama.livasun import Livasun, LivasunConfig
+
+    ff = {"kind": "moe", "expert": {"ff": s["ff"]}, "shared": {"ff": s["top"] * s["ff"] // 2},
+          "router": {"experts": s["experts"], "top": s["top"], "scale": 2.0, "groups": {"count": s["groups"], "keep": s["keep_groups"]}}}
+    att = {"type": "attention", "mlp": ff, "mixer": {
+        "heads": s["heads"], "kv_heads": s["kv"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+        "mask": {"size": s["window"]}, "q_temp": {"coef": 0.1, "every": 1024}, "v_mix": True}}
+    mam = {"type": "mamba2", "mlp": ff, "mixer": {"heads": s["m_heads"], "vdim": s["m_vdim"], "state": s["state"], "groups": 1,
+                                                  "norm_groups": 1, "conv": 4}}
+    lin = {"type": "lightning", "mlp": ff, "mixer": {"heads": s["l_heads"], "dim": s["l_dim"], "vdim": s["l_dim"],
+                                                     "decay": [1.0 - 2.0 ** -(2 + 6 * h / s["l_heads"]) for h in range(s["l_heads"])]}}
+    cfg = {"vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+           "layers": [att, mam, lin, dict(att, mlp={"kind": "dense", "ff": s["top"] * s["ff"]})][: s["layers"]]}
+    m = Livasun(LivasunConfig.from_dict(cfg), dtype=dtype, device=device)
+    g = torch.Generator(device=device).manual_seed(0)
+    fixed = {"dt_bias": -1.0, "a_log": 0.0, "skip": 1.0, "correction": -0.1}
+    for n, p in m.named_parameters():
+        leaf = n.rsplit(".", 1)[-1]
+        if p.dim() >= 2 and "conv" not in n:
+            p.copy_((torch.randn(p.shape, generator=g, device=device) / math.sqrt(p.shape[-1])).to(p.dtype))
+        elif p.dim() >= 2:
+            p.copy_(0.3 * torch.randn(p.shape, generator=g, device=device))
+        elif leaf in fixed:
+            p.fill_(fixed[leaf])
+    m.blocks[-1].mix.v_lambda = 0.4
+    return m.eval()
+
+
+def livasun_kernel_table(s, model, device, timer, prompt_len):
+    """The kernels of one layer of each kind alone.  Roofline time = max(flops / tensor peak, bytes / copy bandwidth), flops and
+    bytes counted for the mechanism (one sweep over the visible keys; one update and one read-out of the state per token)."""
+    from torch.nn import functional as F
+
+    from lit_llama.feed_forward import glu_unit, relu_squared_
+    from lit_llama.recurrence import decay_scan, decay_scan_constant
+    from lit_llama.stepping import add_layer_norm
+
+    hbm, tflops, which = peaks()
+    bf = torch.bfloat16
+    rows = []
+
+    def add(name, t, flops, nbytes):
+        roof = max(flops / tflops, nbytes / hbm)
+        rows.append(dict(kernel=name, us=round(t * 1e6, 1), roofline_us=round(roof * 1e6, 2), fraction=round(roof / t, 4)))
+
+    E, H, G, D, W = s["width"], s["heads"], s["kv"], s["dim"], s["window"]
+    att, mam, lin = (next(b for b in reversed(model.blocks) if b.kind == k).mix for k in ("attention", "mamba2", "lightning"))
+    blk = model.blocks[0]
+    sms = torch.cuda.get_device_properties(device).multi_processor_count
+    for T, tag in ((prompt_len, "prefill"), (1, "decode")):
+        pos0 = 0 if T > 1 else prompt_len
+        pos_ids = torch.arange(pos0, pos0 + T, dtype=torch.int32, device=device)
+        model.reset_cache()
+        model._begin(1, prompt_len + 64, True)
+        for t in model.kv_caches:
+            t.normal_()
+        for t in model.states:
+            t.zero_()
+        x = torch.randn((T, E), device=device, dtype=bf)
+        proj = F.linear(x, att.w_in)
+        first = att.values(proj).clone()
+        caches = model.kv_caches[-2:]
+        span = min(W, caches[0].shape[1])
+        splits = 1 if T > 1 else max(1, min(64, (2 * sms) // max(1, (H + 3) // 4), (span + 31) // 32))
+        keys = sum(min(W, p + 1) for p in range(pos0, pos0 + T))
+        add(f"attention {tag} (head norms + temperature + value mix + append + biased attention)",
+            timer(lambda: att.attend(proj, 1, T, pos_ids, caches, None, splits, first_values=first), graph=True), 2.0 * keys * H * 2 * D,
+            2.0 * (min(W + T, pos0 + T) * G * 2 * D + 2 * T * H * D + 2 * T * G * D))
+        ls = lin.spec
+        lp = F.linear(x, lin.w_in)
+        c = lin.cols
+        st_l = torch.zeros((1, ls.heads, ls.dim, ls.vdim), device=device)
+        nst = ls.heads * ls.dim * ls.vdim
+        add(f"decay_scan {tag} (constant decay, with silu)",
+            timer(lambda: decay_scan_constant(lp, c["q"], c["k"], c["v"], lin.decay, True, 1.0, st_l, pos_ids, 1, T, ls.heads, ls.heads,
+                                              ls.dim, ls.vdim), graph=True), 4.0 * T * nst,
+            2.0 * T * ls.heads * (2 * ls.dim + ls.vdim) + 4.0 * T * ls.heads * ls.vdim + 8.0 * nst)
+        ms = mam.spec
+        xbc = torch.randn((T, ms.conv_channels), device=device, dtype=bf)
+        dtv, dec = torch.rand((T, ms.heads), device=device) * 0.5, torch.rand((T, ms.heads), device=device) * 0.1 + 0.9
+        st_m = torch.zeros((1, ms.heads, ms.state, ms.vdim), device=device)
+        gn = ms.groups * ms.state
+        nst = ms.heads * ms.state * ms.vdim
+        add(f"decay_scan {tag} (state space)",
+            timer(lambda: decay_scan(xbc, ms.inner + gn, xbc, ms.inner, xbc, 0, dec, False, dtv, mam.skip, 1.0, st_m, pos_ids, 1, T, ms.heads,
+                                     ms.groups, ms.state, ms.vdim), graph=True), 4.0 * T * nst,
+            2.0 * T * ms.conv_channels + 4.0 * T * (2 * ms.heads + ms.inner) + 8.0 * nst)
+        pm = F.linear(x, mam.w_in)
+        cst = model.states[0]
+        add(f"short_conv {tag}", timer(lambda: mam.conv(pm, ms.inner, cst, pos_ids, 1, T, bf, silu=True), graph=True), 0.0,
+            T * ms.conv_channels * 4.0)
+        gated_norm_row(f"gated norm {tag} (state space)", torch.randn((T, ms.inner), device=device), pm, 0, mam.norm, False, ms.norm_groups,
+                       True, False, timer, add)
+        gated_norm_row(f"gated norm {tag} (linear attention)", torch.randn((T, ls.heads * ls.vdim), device=device), lp, c["g"], lin.norm,
+                       False, 1, False, True, timer, add)
+        xs, a0, h = torch.randn((T, E), device=device), torch.randn((T, E), device=device, dtype=bf), torch.empty((T, E), device=device, dtype=bf)
+        add(f"add + layer norm {tag}", timer(lambda: add_layer_norm(xs, a0, 1.0, blk.norm1.w, blk.norm1.b, 1e-5, h, bf), graph=True), 0.0,
+            T * E * (4 + 4 + 2 + 2))
+        moe_rows(blk.mlp, x, timer, add, tag)
+        sf = blk.mlp.spec.shared_ff
+        hs = torch.randn((T, sf), device=device, dtype=bf)
+        add(f"relu^2 {tag} (always-on expert)", timer(lambda: relu_squared_(hs), graph=True), 0.0, T * sf * 4)
+        ff = s["top"] * s["ff"]
+        gu = torch.randn((T, 2 * ff), device=device, dtype=bf)
+        add(f"silu-gated unit {tag}", timer(lambda: glu_unit(gu, ff), graph=True), 0.0, T * ff * 6)
+    return rows, which
+
+
+def run_livasun(args):
+    import sys
+
+    sys.path.insert(0, str(ROOT))
+    from __graft_entry__ import build
+
+    build()
+    device = torch.device("cuda", 0)
+    torch.cuda.set_device(device)
+    timer = Timer(device)
+    prompt_len = 2048
+    out = {"family": "livasun", "beside": "bededra", "dtype": "bf16", "data": "synthetic (random weights)", "prompt_len": prompt_len,
+           "batch": 1, "l2": "256 MB written between timed iterations", "sizes": {}}
+    for name in [n for n in LIVASUN_SIZES if not getattr(args, "size", None) or n == args.size]:
+        s = LIVASUN_SIZES[name]
+        with torch.no_grad():
+            m = livasun_model(s, device)
+            pre, dec = end_to_end(m, timer, prompt_len, device, prompt_len + 64)
+            rows, which = livasun_kernel_table(s, m, device, timer, prompt_len)
+            del m
+            torch.cuda.empty_cache()
+            bs = dict(BEDEDRA_SIZES[name], layers=s["layers"])
+            bed = bededra_model(bs, device)
+            bpre, bdec = end_to_end(bed, timer, prompt_len, device, prompt_len + 64)
+            brows, _ = bededra_kernel_table(bs, bed, device, timer, prompt_len)
+            del bed
+            torch.cuda.empty_cache()
+        out["sizes"][name] = {"config": s, "livasun": {"prefill_tokens_per_s": round(pre), "decode_tokens_per_s": round(dec, 1)},
+                              "bededra_same_width": {"prefill_tokens_per_s": round(bpre), "decode_tokens_per_s": round(bdec, 1)},
+                              "kernels": rows, "bededra_kernels": brows, "roofline": f"of {which}"}
+    print(json.dumps(out))
+    return 0
+
+
 def run(args):
     import sys
+
+    if args.family == "livasun":
+        return run_livasun(args)
 
     if args.family == "bededra":
         return run_bededra(args)

@@ -403,12 +403,12 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, int y_gs, c
 }
 
 // The same for long parts (a whole row of heads normed together): a block per (row, part), the gated numbers of the first sweep
-// kept in shared memory.
-template <typename TA>
+// kept in shared memory.  V numbers at a time per thread (4: rows and parts on 4-number boundaries).
+template <typename TA, int V>
 __global__ void gated_group_norm_wide_kernel(const float* __restrict__ y, const TA* __restrict__ gate, int gate_stride,
                                              const float* __restrict__ w, int w_shared, float eps, int gate_first, int gate_sigmoid,
                                              TA* __restrict__ out, int gs) {
-  extern __shared__ float ggn_row[];
+  extern __shared__ __align__(16) float ggn_row[];
   __shared__ float red[32];
   const size_t m = blockIdx.y;
   const int g = blockIdx.x, groups = gridDim.x;
@@ -417,13 +417,49 @@ __global__ void gated_group_norm_wide_kernel(const float* __restrict__ y, const 
   const float* wr = w + (w_shared ? 0 : (size_t)g * gs);
   TA* orow = out + (m * groups + g) * gs;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < gs; i += blockDim.x) {
-    const float z = dt<TA>::ld(gr, i), sg = (gate_sigmoid ? 1.f : z) / (1.f + expf(-z)), v = yr[i];
-    ss += gate_first ? (v * sg) * (v * sg) : v * v;
-    ggn_row[i] = v * sg;
+  auto gated = [&](float v, float z) {
+    const float t = v * (gate_sigmoid ? 1.f : z) / (1.f + expf(-z));
+    ss += gate_first ? t * t : v * v;
+    return t;
+  };
+#pragma unroll 4
+  for (int i = threadIdx.x * V; i < gs; i += blockDim.x * V) {
+    if constexpr (V == 4) {
+      const float4 v = *(const float4*)(yr + i), z = ld4<TA>(gr + i);
+      *(float4*)(ggn_row + i) = make_float4(gated(v.x, z.x), gated(v.y, z.y), gated(v.z, z.z), gated(v.w, z.w));
+    } else {
+      ggn_row[i] = gated(yr[i], dt<TA>::ld(gr, i));
+    }
   }
   const float k = 1.f / sqrtf(block_sum(ss, red) / (float)gs + eps);
-  for (int i = threadIdx.x; i < gs; i += blockDim.x) dt<TA>::st(orow, i, ggn_row[i] * k * wr[i]);
+#pragma unroll 4
+  for (int i = threadIdx.x * V; i < gs; i += blockDim.x * V) {
+    if constexpr (V == 4) {
+      const float4 t = *(const float4*)(ggn_row + i), wv = *(const float4*)(wr + i);
+      st4<TA>(orow + i, make_float4(t.x * k * wv.x, t.y * k * wv.y, t.z * k * wv.z, t.w * k * wv.w));
+    } else {
+      dt<TA>::st(orow, i, ggn_row[i] * k * wr[i]);
+    }
+  }
+}
+
+template <typename TA>
+static int gated_group_norm_wide_launch(const float* y, const void* gate, int gate_stride, const float* w, int w_shared, float eps,
+                                        int groups, int gate_first, int gate_sigmoid, void* out, int rows, int gs, cudaStream_t st) {
+  const bool vec = ((gs | gate_stride) & 3) == 0 && (((uintptr_t)y | (uintptr_t)w | (uintptr_t)out | (uintptr_t)gate) & (4 * sizeof(TA) - 1)) == 0 &&
+                   (((uintptr_t)y | (uintptr_t)w) & 15) == 0;
+  // few blocks: a thread's share of the row is what the launch takes
+  int nt = (long long)rows * groups < 2 * sm_count() ? 1024 : 256;
+  while (nt > 64 && nt * (vec ? 4 : 1) > gs) nt /= 2;
+  const size_t smem = (size_t)gs * sizeof(float);
+#define LL_GGN(V)                                                                                                                     \
+  gated_group_norm_wide_kernel<TA, V><<<dim3(groups, rows), nt, smem, st>>>(y, (const TA*)gate, gate_stride, w, w_shared, eps, gate_first, \
+                                                                            gate_sigmoid, (TA*)out, gs)
+  if (vec) LL_GGN(4);
+  else LL_GGN(1);
+#undef LL_GGN
+  LL_LAUNCH_OK("gated_group_norm_wide_kernel");
+  return LL_OK;
 }
 
 // in place: relu(v)^2
@@ -694,20 +730,13 @@ int ll_gated_group_norm(const float* y, int y_gs, const float* stab, const void*
   cudaStream_t st = (cudaStream_t)stream;
   const int gs = C / groups;
   if (gs >= 256 && gs <= 12288 && !stab && y_gs == gs && rows <= 65535) {
-    const int nt = gs >= 1024 ? 256 : 128;
-    const size_t smem = (size_t)gs * sizeof(float);
     if (act_dtype == LL_F32)
-      gated_group_norm_wide_kernel<float><<<dim3(groups, rows), nt, smem, st>>>(y, (const float*)gate, gate_stride, w, w_shared, eps,
-                                                                               gate_first, gate_sigmoid, (float*)out, gs);
-    else if (act_dtype == LL_BF16)
-      gated_group_norm_wide_kernel<__nv_bfloat16><<<dim3(groups, rows), nt, smem, st>>>(
-          y, (const __nv_bfloat16*)gate, gate_stride, w, w_shared, eps, gate_first, gate_sigmoid, (__nv_bfloat16*)out, gs);
-    else {
-      set_error("gated_group_norm: unsupported dtype %d", act_dtype);
-      return LL_ERR_UNSUPPORTED;
-    }
-    LL_LAUNCH_OK("gated_group_norm_wide_kernel");
-    return LL_OK;
+      return gated_group_norm_wide_launch<float>(y, gate, gate_stride, w, w_shared, eps, groups, gate_first, gate_sigmoid, out, rows, gs, st);
+    if (act_dtype == LL_BF16)
+      return gated_group_norm_wide_launch<__nv_bfloat16>(y, gate, gate_stride, w, w_shared, eps, groups, gate_first, gate_sigmoid, out, rows,
+                                                         gs, st);
+    set_error("gated_group_norm: unsupported dtype %d", act_dtype);
+    return LL_ERR_UNSUPPORTED;
   }
   const int threads = groups >= 8 ? 256 : groups >= 4 ? 128 : 32 * groups;
   if (act_dtype == LL_F32)

@@ -528,6 +528,16 @@ LL_API int ll_decay_scan(const void* q, int q_stride, const void* k, int k_strid
 LL_API int ll_decay_scan_constant(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, int dtype,
                                   const float* a, int act_silu, float qs, float* state, const int32_t* pos_ids, float* y, int B, int T,
                                   int H, int qk_heads, int n, int p, ll_stream stream);
+/* The same recurrence for bf16 prompts in chunks of 64 tokens on tensor cores (csrc/decay_chunk.cu): decays in (0, 1] (0 counts as
+ * e^-10000), a fp32 [B*T][H], or [H] when a_constant; act_silu as above; ks, skip as in ll_decay_scan.  ll_decay_chunked_supported:
+ * bf16, T >= 64, n <= 128 and p in multiples of 8, strides too; q, k, v, state, y and scratch
+ * (ll_decay_chunked_scratch_bytes) on 16-byte boundaries. */
+LL_API int ll_decay_chunked_supported(int dtype, int T, int n, int p, int q_stride, int k_stride, int v_stride);
+LL_API size_t ll_decay_chunked_scratch_bytes(int B, int T, int H, int n, int p);
+LL_API int ll_decay_chunked(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, int dtype,
+                            const float* a, int a_constant, int act_silu, const float* ks, const float* skip, float qs, float* state,
+                            const int32_t* pos_ids, float* y, int B, int T, int H, int qk_heads, int n, int p, float* scratch,
+                            ll_stream stream);
 /* Exponential gates with a running stabiliser, per (b, h): li = cap(raw_i + bias_i[h]), lf = logsigmoid(cap(raw_f + bias_f[h])),
  * cap(z) = c tanh(z / c) (c <= 0: none); mx_t = max(lf_t + mx_(t-1), li_t) with mx carried in mstate fp32 [B][H] (0 when
  * pos_ids[0] == 0); keep = exp(lf + mx_(t-1) - mx_t), take = exp(li - mx_t), stab = mx_t   (fp32 [B*T][H] each). */

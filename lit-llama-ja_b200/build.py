@@ -22,9 +22,9 @@ FLAGS = [
 # for that family, and no more.  quant_pack carries the library's error plumbing and version.
 FAMILY_SOURCES = {
     "Lepalorn": ["quant_pack", "decode_ops", "sampling", "residual_ops", "latent_attn", "moe_ops", "moe_gemm_tc"],
-    "Bededra": ["quant_pack", "residual_ops", "short_conv", "decay_scan", "window_attn", "moe_ops", "moe_gemm_tc"],
+    "Bededra": ["quant_pack", "residual_ops", "short_conv", "decay_scan", "decay_chunk", "window_attn", "moe_ops", "moe_gemm_tc"],
     "Tebodra": ["quant_pack", "residual_ops", "short_conv", "decay_scan", "rotary_attn"],
-    "Livasun": ["quant_pack", "residual_ops", "short_conv", "decay_scan", "rotary_attn", "moe_ops", "moe_gemm_tc"],
+    "Livasun": ["quant_pack", "residual_ops", "short_conv", "decay_scan", "decay_chunk", "rotary_attn", "moe_ops", "moe_gemm_tc"],
     "Bumulix": ["quant_pack", "residual_ops", "rotary_attn", "latent_attn"],
 }
 

@@ -62,6 +62,12 @@ template <> struct dt<__half> {
   static __device__ __forceinline__ float rd(float v) { return __half2float(__float2half_rn(v)); }
 };
 
+// silu, rounded to the activation dtype.  bf16: from one fast exponential and one fast division, whose error lies far below the
+// rounding; the kernels that form it all do so here, so that they agree bit for bit.
+template <typename T> __device__ __forceinline__ float silu_act(float x);
+template <> __device__ __forceinline__ float silu_act<float>(float x) { return x / (1.f + expf(-x)); }
+template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float x) { return bf16r(__fdividef(x, 1.f + __expf(-x))); }
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

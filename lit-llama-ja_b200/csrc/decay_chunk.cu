@@ -1,0 +1,382 @@
+// The linear recurrence of decay_scan.cu for prompts in bf16, on tensor cores: with one decay per head and token (or one constant
+// per head) the walk over tokens can be cut into chunks of 64 whose work is matrix products.  Per (sequence, head), G_t the sum of
+// log a over the chunk up to token t:
+//
+//   collect   D_c = sum_s e^(G_last - G_s) (ks_s k_s) v_s^T             what a chunk adds to the state      (a block per chunk)
+//   pass      S_c = e^(G_last) S_(c-1) + D_c                            the state before every chunk        (fp32, element by element)
+//   read      y_t = qs ( sum_(s <= t) e^(G_t - G_s) ks_s (q_t.k_s) v_s + e^(G_t) S_(c-1)^T q_t ) + skip v_t     (a block per chunk)
+//
+// q, k and v are bf16 as they stand, so only the fp32 factors have to be split for the bf16 tensor cores (fp32 accumulation):
+// e^(..) ks k enters D as three bf16 terms (24 bits: what is carried on is as exact as the walk's fp32), the chunk's weights and
+// the state meet v and q as two terms (16 bits, the sum of both products in fp32).  Sums of log a are formed in fp64, so that the
+// difference of two of them keeps its digits whatever lies before it in the chunk.  The state handed on is fp32.
+#include "common.cuh"
+
+namespace llb {
+
+constexpr int DC_L = 64, DC_PT = 64, DC_THREADS = 128;       // tokens of a chunk, value columns of a block
+constexpr int DC_LV = DC_PT + 8;
+constexpr double DC_LOG_MIN = -1e4;                          // log of a decay of zero: e^-10000 is zero in fp32
+
+__device__ __forceinline__ void dc_ldmatrix(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void dc_ldmatrix_trans(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ uint32_t dc_pack(float a, float b) { return (uint32_t)f32_to_bf16_bits(a) | ((uint32_t)f32_to_bf16_bits(b) << 16); }
+// x as bf16 terms: the first of (a, b) packed, the rest left in a and b
+__device__ __forceinline__ uint32_t dc_term(float& a, float& b) {
+  const float ha = bf16r(a), hb = bf16r(b);
+  a -= ha, b -= hb;
+  return (uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(ha)) | ((uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(hb)) << 16);
+}
+template <bool SILU>
+__device__ __forceinline__ uint32_t dc_in2(uint32_t u) {
+  if (!SILU) return u;
+  return dc_pack(silu_act<__nv_bfloat16>(bf16_bits_to_f32(u & 0xffffu)), silu_act<__nv_bfloat16>(bf16_bits_to_f32(u >> 16)));
+}
+template <bool SILU>
+__device__ __forceinline__ uint4 dc_in8(uint4 u) {
+  return make_uint4(dc_in2<SILU>(u.x), dc_in2<SILU>(u.y), dc_in2<SILU>(u.z), dc_in2<SILU>(u.w));
+}
+
+// G[t] = sum over the chunk's tokens up to t of log a (tokens past the end: a = 1), by the first warp, two tokens a lane
+__device__ __forceinline__ void dc_log_sums(const float* __restrict__ a, int a_row, int h, size_t m0, int len, double* G) {
+  if (threadIdx.x >= 32) return;
+  const int lane = threadIdx.x;
+  double v[2];
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int t = 2 * lane + e;
+    v[e] = t < len ? fmax((double)logf(a[(m0 + t) * a_row + h]), DC_LOG_MIN) : 0.0;
+  }
+  double incl = v[0] + v[1];
+#pragma unroll
+  for (int d = 1; d < 32; d <<= 1) {
+    const double o = __shfl_up_sync(0xffffffffu, incl, d);
+    if (lane >= d) incl += o;
+  }
+  G[2 * lane] = incl - v[1];
+  G[2 * lane + 1] = incl;
+}
+
+// grid (chunks * p tiles, H, B): D_c into dst[((b * H + h) * chunks + c)][n][p], e^(G_last) into total[(b * H + h) * chunks + c].
+// NP: n rounded up to 16, 32, 64 or 128.
+template <int NP, bool SILU>
+__global__ void __launch_bounds__(DC_THREADS) decay_collect_kernel(const __nv_bfloat16* __restrict__ k, int k_stride,
+                                                                   const __nv_bfloat16* __restrict__ v, int v_stride,
+                                                                   const float* __restrict__ a, int a_row, const float* __restrict__ ks,
+                                                                   float* __restrict__ dst, float* __restrict__ total, int Tn, int H,
+                                                                   int qk_heads, int n, int p, int ptiles) {
+  constexpr int LK = NP + 8;
+  extern __shared__ __align__(16) unsigned char dc_smem[];
+  __nv_bfloat16* Ks = (__nv_bfloat16*)dc_smem;                // [3 terms][64][LK]
+  __nv_bfloat16* Vs = Ks + 3 * DC_L * LK;                     // [64][LV]
+  __shared__ double G[DC_L];
+  __shared__ float wgt[DC_L];
+  const int c = blockIdx.x / ptiles, p0 = (blockIdx.x - c * ptiles) * DC_PT, h = blockIdx.y, b = blockIdx.z, g = h / (H / qk_heads);
+  const int chunks = gridDim.x / ptiles, t0 = c * DC_L, len = min(DC_L, Tn - t0), tid = threadIdx.x;
+  const size_t m0 = (size_t)b * Tn + t0;
+  const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
+  dc_log_sums(a, a_row, h, m0, len, G);
+  for (int i = tid; i < DC_L * (DC_PT / 8); i += DC_THREADS) {
+    const int s = i / (DC_PT / 8), ch = (i % (DC_PT / 8)) * 8;
+    uint4 u = zero4;
+    if (s < len && p0 + ch < p) u = dc_in8<SILU>(*(const uint4*)(v + (m0 + s) * v_stride + (size_t)h * p + p0 + ch));
+    *(uint4*)&Vs[s * DC_LV + ch] = u;
+  }
+  __syncthreads();
+  if (tid < DC_L) wgt[tid] = tid < len ? expf((float)(G[DC_L - 1] - G[tid])) * (ks ? ks[(m0 + tid) * H + h] : 1.f) : 0.f;
+  if (tid == 0 && p0 == 0) total[((size_t)b * H + h) * chunks + c] = expf((float)G[DC_L - 1]);
+  __syncthreads();
+  for (int i = tid; i < DC_L * (NP / 8); i += DC_THREADS) {
+    const int s = i / (NP / 8), ch = (i % (NP / 8)) * 8;
+    uint4 u = zero4;
+    if (s < len && ch < n) u = dc_in8<SILU>(*(const uint4*)(k + (m0 + s) * k_stride + (size_t)g * n + ch));
+    const float w = wgt[s];
+    const uint32_t in[4] = {u.x, u.y, u.z, u.w};
+    uint32_t out[3][4];
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      float x0 = bf16_bits_to_f32(in[q] & 0xffffu) * w, x1 = bf16_bits_to_f32(in[q] >> 16) * w;
+      out[0][q] = dc_term(x0, x1);
+      out[1][q] = dc_term(x0, x1);
+      out[2][q] = dc_pack(x0, x1);
+    }
+#pragma unroll
+    for (int z = 0; z < 3; ++z) *(uint4*)&Ks[(z * DC_L + s) * LK + ch] = make_uint4(out[z][0], out[z][1], out[z][2], out[z][3]);
+  }
+  __syncthreads();
+  const int warp = tid >> 5, lane = tid & 31;
+  float* D = dst + (((size_t)b * H + h) * chunks + c) * (size_t)n * p;
+#pragma unroll 1
+  for (int mt = warp; mt < NP / 16; mt += DC_THREADS / 32) {
+    if (mt * 16 >= n) break;
+    float acc[DC_PT / 8][4];
+#pragma unroll
+    for (int f = 0; f < DC_PT / 8; ++f) acc[f][0] = acc[f][1] = acc[f][2] = acc[f][3] = 0.f;
+#pragma unroll
+    for (int st = 0; st < DC_L / 16; ++st) {
+      uint32_t bf[DC_PT / 16][4];
+#pragma unroll
+      for (int d = 0; d < DC_PT / 16; ++d)
+        dc_ldmatrix_trans(bf[d], &Vs[(st * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * DC_LV + d * 16 + (lane >> 4) * 8]);
+#pragma unroll
+      for (int z = 2; z >= 0; --z) {                          // the smallest term first
+        uint32_t af[4];
+        dc_ldmatrix_trans(af, &Ks[(z * DC_L + st * 16 + (lane & 7) + (lane >> 4) * 8) * LK + mt * 16 + ((lane >> 3) & 1) * 8]);
+#pragma unroll
+        for (int d = 0; d < DC_PT / 16; ++d) {
+          mma_bf16_16816(acc[2 * d], af[0], af[1], af[2], af[3], bf[d][0], bf[d][1]);
+          mma_bf16_16816(acc[2 * d + 1], af[0], af[1], af[2], af[3], bf[d][2], bf[d][3]);
+        }
+      }
+    }
+#pragma unroll
+    for (int f = 0; f < DC_PT / 8; ++f)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int i = mt * 16 + (lane >> 2) + e * 8, col = p0 + f * 8 + (lane & 3) * 2;
+        if (i < n && col < p) *(float2*)(D + (size_t)i * p + col) = make_float2(acc[f][2 * e], acc[f][2 * e + 1]);
+      }
+  }
+}
+
+// Per (sequence, head), four neighbouring elements of the state a thread: D_c is replaced by the state before chunk c, the state
+// after the last chunk goes back to `state`.
+__global__ void __launch_bounds__(128) decay_pass_kernel(float* __restrict__ chunk_state, const float* __restrict__ total,
+                                                         float* __restrict__ state, const int32_t* __restrict__ pos_ids, int chunks,
+                                                         int np4) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= np4) return;
+  const size_t bh = blockIdx.y;
+  float4* D = (float4*)chunk_state + bh * chunks * np4 + i;
+  float4* S = (float4*)state + bh * np4 + i;
+  const float* tot = total + bh * chunks;
+  float4 s = pos_ids[0] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *S;
+  constexpr int AHEAD = 8;                                    // chunks whose loads are in flight together
+  for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+    float4 d[AHEAD];
+    float w[AHEAD];
+#pragma unroll
+    for (int j = 0; j < AHEAD; ++j)
+      if (c0 + j < chunks) d[j] = D[(size_t)(c0 + j) * np4], w[j] = tot[c0 + j];
+#pragma unroll
+    for (int j = 0; j < AHEAD; ++j)
+      if (c0 + j < chunks) {
+        D[(size_t)(c0 + j) * np4] = s;
+        s = make_float4(w[j] * s.x + d[j].x, w[j] * s.y + d[j].y, w[j] * s.z + d[j].z, w[j] * s.w + d[j].w);
+      }
+  }
+  *S = s;
+}
+
+// grid (chunks * p tiles, H, B).  A warp owns 16 consecutive tokens; its queries come from global memory straight into fragments.
+template <int NP, bool SILU>
+__global__ void __launch_bounds__(DC_THREADS, 3) decay_read_kernel(
+    const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ k, int k_stride, const __nv_bfloat16* __restrict__ v,
+    int v_stride, const float* __restrict__ a, int a_row, const float* __restrict__ ks, const float* __restrict__ skip, float qs,
+    const float* __restrict__ chunk_state, const int32_t* __restrict__ pos_ids, float* __restrict__ y, int Tn, int H, int qk_heads, int n,
+    int p, int ptiles) {
+  constexpr int LK = NP + 8;
+  extern __shared__ __align__(16) unsigned char dc_smem[];
+  __nv_bfloat16* Ks = (__nv_bfloat16*)dc_smem;                // [64][LK]
+  __nv_bfloat16* Vs = Ks + DC_L * LK;                         // [64][LV]
+  __nv_bfloat16* Ss = Vs + DC_L * DC_LV;                      // [2 terms][NP][LV]
+  __shared__ double G[DC_L];
+  __shared__ float kw[DC_L];
+  const int c = blockIdx.x / ptiles, p0 = (blockIdx.x - c * ptiles) * DC_PT, h = blockIdx.y, b = blockIdx.z, g = h / (H / qk_heads);
+  const int chunks = gridDim.x / ptiles, t0 = c * DC_L, len = min(DC_L, Tn - t0);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const size_t m0 = (size_t)b * Tn + t0;
+  const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
+  const bool has_state = c > 0 || pos_ids[0] != 0;
+  for (int i = tid; i < DC_L * (NP / 8); i += DC_THREADS) {
+    const int s = i / (NP / 8), ch = (i % (NP / 8)) * 8;
+    uint4 u = zero4;
+    if (s < len && ch < n) u = dc_in8<SILU>(*(const uint4*)(k + (m0 + s) * k_stride + (size_t)g * n + ch));
+    *(uint4*)&Ks[s * LK + ch] = u;
+  }
+  for (int i = tid; i < DC_L * (DC_PT / 8); i += DC_THREADS) {
+    const int s = i / (DC_PT / 8), ch = (i % (DC_PT / 8)) * 8;
+    uint4 u = zero4;
+    if (s < len && p0 + ch < p) u = dc_in8<SILU>(*(const uint4*)(v + (m0 + s) * v_stride + (size_t)h * p + p0 + ch));
+    *(uint4*)&Vs[s * DC_LV + ch] = u;
+  }
+  if (has_state) {
+    const float* S = chunk_state + (((size_t)b * H + h) * chunks + c) * (size_t)n * p;
+#pragma unroll 4
+    for (int i = tid; i < NP * (DC_PT / 4); i += DC_THREADS) {
+      const int r = i / (DC_PT / 4), col = (i % (DC_PT / 4)) * 4;
+      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (r < n && p0 + col < p) f = *(const float4*)(S + (size_t)r * p + p0 + col);
+      const uint32_t h0 = dc_term(f.x, f.y), h1 = dc_term(f.z, f.w);
+      *(uint2*)&Ss[r * DC_LV + col] = make_uint2(h0, h1);
+      *(uint2*)&Ss[(NP + r) * DC_LV + col] = make_uint2(dc_pack(f.x, f.y), dc_pack(f.z, f.w));
+    }
+  }
+  if (tid < DC_L) kw[tid] = tid < len ? (ks ? ks[(m0 + tid) * H + h] : 1.f) * qs : 0.f;
+  dc_log_sums(a, a_row, h, m0, len, G);
+  // query fragments: rows (lane / 4) and + 8 of the warp's 16, columns (lane % 4) * 2 and + 8 of every 16
+  uint32_t qf[NP / 16][4];
+  const int r0 = warp * 16 + (lane >> 2);
+#pragma unroll
+  for (int kk = 0; kk < NP / 16; ++kk)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = r0 + (e & 1) * 8, col = kk * 16 + (lane & 3) * 2 + (e >> 1) * 8;
+      qf[kk][e] = (r < len && col < n) ? dc_in2<SILU>(*(const uint32_t*)(q + (m0 + r) * q_stride + (size_t)g * n + col)) : 0u;
+    }
+  __syncthreads();
+  if (warp * 16 >= len) return;
+  float o[DC_PT / 8][4];
+#pragma unroll
+  for (int f = 0; f < DC_PT / 8; ++f) o[f][0] = o[f][1] = o[f][2] = o[f][3] = 0.f;
+  const double g0 = G[r0], g1 = G[r0 + 8];
+  if (has_state) {
+#pragma unroll
+    for (int kk = 0; kk < NP / 16; ++kk)
+#pragma unroll
+      for (int z = 1; z >= 0; --z)
+#pragma unroll
+        for (int d = 0; d < DC_PT / 16; ++d) {
+          uint32_t bf[4];
+          dc_ldmatrix_trans(bf, &Ss[(z * NP + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * DC_LV + d * 16 + (lane >> 4) * 8]);
+          mma_bf16_16816(o[2 * d], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], bf[0], bf[1]);
+          mma_bf16_16816(o[2 * d + 1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], bf[2], bf[3]);
+        }
+    const float e0 = expf((float)g0) * qs, e1 = expf((float)g1) * qs;
+#pragma unroll
+    for (int f = 0; f < DC_PT / 8; ++f) o[f][0] *= e0, o[f][1] *= e0, o[f][2] *= e1, o[f][3] *= e1;
+  }
+#pragma unroll
+  for (int st = 0; st < DC_L / 16; ++st) {                    // 16 keys at a time, none that lie after all of the warp's tokens
+    if (st > warp) break;
+    float sc[2][4];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+#pragma unroll
+    for (int kk = 0; kk < NP / 16; ++kk) {
+      uint32_t bf[4];
+      dc_ldmatrix(bf, &Ks[(st * 16 + (lane & 7) + (lane >> 4) * 8) * LK + kk * 16 + ((lane >> 3) & 1) * 8]);
+      mma_bf16_16816(sc[0], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], bf[0], bf[1]);
+      mma_bf16_16816(sc[1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], bf[2], bf[3]);
+    }
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int s = st * 16 + j * 8 + (lane & 3) * 2 + (e & 1), r = r0 + (e >> 1) * 8;
+        sc[j][e] = s <= r ? sc[j][e] * (expf((float)((e >> 1 ? g1 : g0) - G[s])) * kw[s]) : 0.f;
+      }
+    uint32_t ah[4], al[4];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      ah[2 * j] = dc_term(sc[j][0], sc[j][1]), al[2 * j] = dc_pack(sc[j][0], sc[j][1]);
+      ah[2 * j + 1] = dc_term(sc[j][2], sc[j][3]), al[2 * j + 1] = dc_pack(sc[j][2], sc[j][3]);
+    }
+#pragma unroll
+    for (int d = 0; d < DC_PT / 16; ++d) {
+      uint32_t bf[4];
+      dc_ldmatrix_trans(bf, &Vs[(st * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * DC_LV + d * 16 + (lane >> 4) * 8]);
+      mma_bf16_16816(o[2 * d], al[0], al[1], al[2], al[3], bf[0], bf[1]);
+      mma_bf16_16816(o[2 * d + 1], al[0], al[1], al[2], al[3], bf[2], bf[3]);
+      mma_bf16_16816(o[2 * d], ah[0], ah[1], ah[2], ah[3], bf[0], bf[1]);
+      mma_bf16_16816(o[2 * d + 1], ah[0], ah[1], ah[2], ah[3], bf[2], bf[3]);
+    }
+  }
+  const float sk = skip ? skip[h] : 0.f;
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int r = r0 + e * 8;
+    if (r >= len) continue;
+    float* yr = y + (m0 + r) * (size_t)H * p + (size_t)h * p + p0;
+#pragma unroll
+    for (int f = 0; f < DC_PT / 8; ++f) {
+      const int col = f * 8 + (lane & 3) * 2;
+      if (p0 + col >= p) continue;
+      float v0 = o[f][2 * e], v1 = o[f][2 * e + 1];
+      if (skip) {
+        v0 += sk * __bfloat162float(Vs[r * DC_LV + col]);
+        v1 += sk * __bfloat162float(Vs[r * DC_LV + col + 1]);
+      }
+      *(float2*)(yr + col) = make_float2(v0, v1);
+    }
+  }
+}
+
+template <int NP, bool SILU>
+static int decay_chunked_launch(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const float* a,
+                                int a_row, const float* ks, const float* skip, float qs, float* state, const int32_t* pos_ids, float* y,
+                                int B, int Tn, int H, int qk_heads, int n, int p, float* scratch, cudaStream_t st) {
+  const int chunks = (Tn + DC_L - 1) / DC_L, ptiles = (p + DC_PT - 1) / DC_PT, np4 = n * p / 4;
+  float* chunk_state = scratch;
+  float* total = scratch + (size_t)B * H * chunks * n * p;
+  const dim3 grid(chunks * ptiles, H, B);
+  constexpr int smem_c = (3 * DC_L * (NP + 8) + DC_L * DC_LV) * 2, smem_r = (DC_L * (NP + 8) + DC_L * DC_LV + 2 * NP * DC_LV) * 2;
+  static bool sized = false;
+  if (!sized) {
+    LL_CUDA(cudaFuncSetAttribute(decay_collect_kernel<NP, SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_c));
+    LL_CUDA(cudaFuncSetAttribute(decay_read_kernel<NP, SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_r));
+    sized = true;
+  }
+  typedef const __nv_bfloat16* in_t;
+  decay_collect_kernel<NP, SILU><<<grid, DC_THREADS, smem_c, st>>>((in_t)k, k_stride, (in_t)v, v_stride, a, a_row, ks, chunk_state, total, Tn, H,
+                                                                  qk_heads, n, p, ptiles);
+  LL_LAUNCH_OK("decay_collect_kernel");
+  decay_pass_kernel<<<dim3((np4 + 127) / 128, B * H), 128, 0, st>>>(chunk_state, total, state, pos_ids, chunks, np4);
+  LL_LAUNCH_OK("decay_pass_kernel");
+  decay_read_kernel<NP, SILU><<<grid, DC_THREADS, smem_r, st>>>((in_t)q, q_stride, (in_t)k, k_stride, (in_t)v, v_stride, a, a_row, ks, skip, qs,
+                                                               chunk_state, pos_ids, y, Tn, H, qk_heads, n, p, ptiles);
+  LL_LAUNCH_OK("decay_read_kernel");
+  return LL_OK;
+}
+
+}  // namespace llb
+
+using namespace llb;
+
+extern "C" {
+
+int ll_decay_chunked_supported(int dtype, int T, int n, int p, int q_stride, int k_stride, int v_stride) {
+  return dtype == LL_BF16 && T >= DC_L && n % 8 == 0 && n <= 128 && p % 8 == 0 && ((q_stride | k_stride | v_stride) & 7) == 0;
+}
+
+size_t ll_decay_chunked_scratch_bytes(int B, int T, int H, int n, int p) {
+  const size_t chunks = (T + DC_L - 1) / DC_L;
+  return (size_t)B * H * chunks * ((size_t)n * p + 1) * sizeof(float);
+}
+
+int ll_decay_chunked(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, int dtype, const float* a,
+                     int a_constant, int act_silu, const float* ks, const float* skip, float qs, float* state, const int32_t* pos_ids,
+                     float* y, int B, int T, int H, int qk_heads, int n, int p, float* scratch, ll_stream stream) {
+  LL_CHECK_ARG(q && k && v && a && state && pos_ids && y && scratch, "decay_chunked: null pointer");
+  LL_CHECK_ARG(B >= 0 && T >= 0 && H > 0 && qk_heads > 0 && H % qk_heads == 0 && n > 0 && p > 0, "bad decay_chunked arguments");
+  if (B == 0 || T == 0) return LL_OK;
+  const uintptr_t at = (uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)state | (uintptr_t)y | (uintptr_t)scratch;
+  if (!ll_decay_chunked_supported(dtype, T, n, p, q_stride, k_stride, v_stride) || (at & 15) != 0 || (long long)B * H > 65535) {
+    set_error("decay_chunked: bf16, at least %d tokens, n and p in multiples of 8 (n up to 128), rows on 16-byte boundaries", DC_L);
+    return LL_ERR_UNSUPPORTED;
+  }
+  cudaStream_t st = (cudaStream_t)stream;
+  const int a_row = a_constant ? 0 : H;
+#define LL_DC_S(NP, SILU)                                                                                                              \
+  return decay_chunked_launch<NP, SILU>(q, q_stride, k, k_stride, v, v_stride, a, a_row, ks, skip, qs, state, pos_ids, y, B, T, H, qk_heads, \
+                                        n, p, scratch, st)
+#define LL_DC(NP)                  \
+  if (n <= NP) {                   \
+    if (act_silu) LL_DC_S(NP, true); \
+    LL_DC_S(NP, false);            \
+  }
+  LL_DC(16) LL_DC(32) LL_DC(64) LL_DC(128)
+#undef LL_DC
+#undef LL_DC_S
+  return LL_ERR_UNSUPPORTED;
+}
+
+}  // extern "C"

@@ -32,7 +32,7 @@ __host__ __device__ constexpr int ds_tc(int npad) { return npad <= 64 ? 16 : npa
 template <typename T, bool SILU>
 __device__ __forceinline__ float ds_in(T raw) {
   const float x = dt<T>::ld(&raw, 0);
-  return SILU ? dt<T>::rd(x / (1.f + expf(-x))) : x;
+  return SILU ? silu_act<T>(x) : x;
 }
 
 template <typename T, int NP, int DS_NL, bool PERCH, bool SILU>

@@ -132,6 +132,10 @@ EXPORTS = {
     "ll_decay_scan": ([vp, i32, vp, i32, vp, i32, i32, vp, i32, vp, vp, C.c_float, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp],
                       C.c_int),
     "ll_decay_scan_constant": ([vp, i32, vp, i32, vp, i32, i32, vp, i32, C.c_float, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp], C.c_int),
+    "ll_decay_chunked_supported": ([i32, i32, i32, i32, i32, i32, i32], C.c_int),
+    "ll_decay_chunked_scratch_bytes": ([i32, i32, i32, i32, i32], sz_t),
+    "ll_decay_chunked": ([vp, i32, vp, i32, vp, i32, i32, vp, i32, i32, vp, vp, C.c_float, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, vp],
+                         C.c_int),
     "ll_matrix_memory_gates": ([vp, vp, i32, i32, vp, vp, C.c_float, vp, vp, vp, vp, vp, i32, i32, i32, vp], C.c_int),
     "ll_qk_rotary_append": ([vp, i32, vp, i32, vp, i32, i32, vp, vp, C.c_float, vp, i32, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32,
                              i32, vp], C.c_int),

@@ -17,11 +17,14 @@
       q, k, v = silu(W_q h), silu(W_k h), silu(W_v h);  S_t = decay_h S_(t-1) + k_t v_t^T;  o_t = S_t^T q_t
       out = W_o ( rmsnorm(all heads together) * w * sigmoid(W_g h) )
 
-Decays, step sizes, the state, the read-out and the norms are fp32; the projections, the short convolution's output and
+Prompts in bfloat16 whose decay is one number per head and token (or a constant per head) run in chunks of 64 tokens on tensor
+cores (csrc/decay_chunk.cu); single tokens, short portions, fp32 and decays per channel walk token by token
+(csrc/decay_scan.cu).  Decays, step sizes, the state, the read-out and the norms are fp32; the projections, the short convolution's output and
 the gates are in the activation dtype.  A sequence at position 0 starts from a zero state whatever its slot holds.
 """
 from __future__ import annotations
 
+import os
 from dataclasses import dataclass
 from typing import List, Tuple
 
@@ -37,11 +40,32 @@ def pad8(n: int) -> int:
     return (n + 7) // 8 * 8
 
 
+USE_CHUNKS = os.environ.get("LLB200_DECAY_CHUNKS", "1") != "0"       # 0: always walk token by token
+
+
+def takes_chunks(T, H, n, p, *slices) -> bool:
+    """Whether a step of ``T`` tokens runs in chunks; ``slices``: (tensor, first column) of q, k and v."""
+    t = [s[0] for s in slices]
+    return (USE_CHUNKS and N.has("ll_decay_chunked")
+            and bool(N.call_ret("ll_decay_chunked_supported", N.dtype_code(t[0].dtype), T, n, p, *[x.stride(0) for x in t]))
+            and all((x.data_ptr() + c * x.element_size()) % 16 == 0 for x, c in slices))
+
+
+def _decay_chunked(q, q_col, k, k_col, v, v_col, decay, constant, silu, kscale, skip, qscale, state, pos_ids, y, B, T, H, qk_heads, n, p):
+    scratch = torch.empty(N.call_ret("ll_decay_chunked_scratch_bytes", B, T, H, n, p) // 4, dtype=torch.float32, device=v.device)
+    N.call("ll_decay_chunked", N.ptr_at(q, q_col), q.stride(0), N.ptr_at(k, k_col), k.stride(0), N.ptr_at(v, v_col), v.stride(0),
+           N.dtype_code(v.dtype), N.ptr(decay), 1 if constant else 0, 1 if silu else 0, N.ptr(kscale), N.ptr(skip), float(qscale),
+           N.ptr(state), N.ptr(pos_ids), N.ptr(y), B, T, H, qk_heads, n, p, N.ptr(scratch), N.stream())
+
+
 def decay_scan(q, q_col, k, k_col, v, v_col, decay, per_channel, kscale, skip, qscale, state, pos_ids, B, T, H, qk_heads, n, p,
                unit_col=False):
     """fp32 ``[B*T, H*p]``: the read-out of the recurrence (see csrc/decay_scan.cu); ``state`` is advanced in place.
     ``unit_col``: the last of the ``p`` columns of every head is the constant 1 (``v`` holds ``p - 1`` per head)."""
     y = torch.empty((B * T, H * p), dtype=torch.float32, device=v.device)
+    if not per_channel and not unit_col and takes_chunks(T, H, n, p, (q, q_col), (k, k_col), (v, v_col)):
+        _decay_chunked(q, q_col, k, k_col, v, v_col, decay, False, False, kscale, skip, qscale, state, pos_ids, y, B, T, H, qk_heads, n, p)
+        return y
     N.call("ll_decay_scan", N.ptr_at(q, q_col), q.stride(0), N.ptr_at(k, k_col), k.stride(0), N.ptr_at(v, v_col), v.stride(0),
            N.dtype_code(v.dtype), N.ptr(decay), 1 if per_channel else 0, N.ptr(kscale), N.ptr(skip), float(qscale), N.ptr(state),
            N.ptr(pos_ids), N.ptr(y), B, T, H, qk_heads, n, p, 1 if unit_col else 0, N.stream())
@@ -52,6 +76,10 @@ def decay_scan_constant(proj, q_col, k_col, v_col, decay, silu, qscale, state, p
     """The same walk with one constant decay per head (``decay`` fp32 ``[H]``) over column slices of one projection output;
     ``silu``: q, k and v pass it as they are read."""
     y = torch.empty((B * T, H * p), dtype=torch.float32, device=proj.device)
+    if takes_chunks(T, H, n, p, (proj, q_col), (proj, k_col), (proj, v_col)):
+        _decay_chunked(proj, q_col, proj, k_col, proj, v_col, decay, True, silu, None, None, qscale, state, pos_ids, y, B, T, H, qk_heads,
+                       n, p)
+        return y
     N.call("ll_decay_scan_constant", N.ptr_at(proj, q_col), proj.stride(0), N.ptr_at(proj, k_col), proj.stride(0), N.ptr_at(proj, v_col),
            proj.stride(0), N.dtype_code(proj.dtype), N.ptr(decay), 1 if silu else 0, float(qscale), N.ptr(state), N.ptr(pos_ids), N.ptr(y),
            B, T, H, qk_heads, n, p, N.stream())

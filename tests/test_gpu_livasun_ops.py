@@ -387,3 +387,88 @@ def test_silu_gated_dense_layer(M, E, ff, dtype):
     f.load(lambda s: dev(W[s]))
     x = rounded(r.randn(M, E), dtype)
     close(f(dev(x, dtype)), O.dense_ff(x, W, ""), TOL[dtype] * 2)
+
+
+# ------------------------------------------------------------------ the recurrences in chunks on tensor cores
+def chunk_case(r, T, H, G, n, p, low=0.5):
+    q, k, v = (bf16(r.randn(T, c)) for c in (G * n, G * n, H * p))
+    a = r.uniform(low, 1.0, (T, H))
+    return q, k, v, a, r.uniform(0.1, 1.5, (T, H)), r.randn(H)
+
+
+def chunk_want(q, k, v, a, ks, skip, qs, H, G, n, p):
+    T = len(q)
+    y = np.zeros((T, H, p))
+    for h in range(H):
+        g, S = h // (H // G), np.zeros((n, p))
+        for t in range(T):
+            S = a[t, h] * S + ks[t, h] * np.outer(k[t, g * n:(g + 1) * n], v[t, h * p:(h + 1) * p])
+            y[t, h] = qs * (S.T @ q[t, g * n:(g + 1) * n]) + skip[h] * v[t, h * p:(h + 1) * p]
+    return y.reshape(T, H * p), S
+
+
+@pytest.mark.parametrize("H,G,n,p", [(2, 1, 8, 8), (4, 2, 16, 24), (3, 3, 40, 64), (2, 1, 64, 72), (2, 2, 128, 136), (6, 1, 104, 16)])
+@pytest.mark.parametrize("low", [0.0, 0.9])
+def test_chunked_recurrence_against_the_walk(H, G, n, p, low):
+    """Chunk edges, last chunks that are not full, a step that begins inside a sequence, decays near zero and near one, a decay of
+    exactly zero in the middle of a chunk; outputs and the state handed on agree with float64 to fp32 accuracy."""
+    import lit_llama.recurrence as R
+
+    r = np.random.RandomState(n + p)
+    T = 300
+    q, k, v, a, ks, skip = chunk_case(r, T, H, G, n, p, low)
+    a[100] = 0.0
+    a[170, 0] = 1e-30
+    want, S = chunk_want(q, k, v, a, ks, skip, 0.5, H, G, n, p)
+    bfl = torch.bfloat16
+    for portions in ([300], [64, 236], [70, 5, 65, 1, 159], [127, 128, 45]):
+        state = torch.full((1, H, n, p), float("nan"), device="cuda")
+        got, at = [], 0
+        for m in portions:
+            ops = [dev(q[at:at + m], bfl), dev(k[at:at + m], bfl), dev(v[at:at + m], bfl)]
+            assert R.takes_chunks(m, H, n, p, *[(o, 0) for o in ops]) == (m >= 64)
+            got.append(R.decay_scan(ops[0], 0, ops[1], 0, ops[2], 0, dev(a[at:at + m]), False, dev(ks[at:at + m]), dev(skip), 0.5, state,
+                                    pos(at, at + m), 1, m, H, G, n, p))
+            at += m
+        close(torch.cat(got), want, 3e-5)                       # (the read-out's weights carry 16 bits)
+        close(state[0, H - 1], S, 2e-6)
+
+
+@pytest.mark.parametrize("H,n,p", [(3, 32, 48), (2, 128, 128), (4, 8, 8)])
+def test_chunked_constant_decay_with_silu(H, n, p, monkeypatch):
+    """The same step walked and in chunks: the same activations bit for bit, so that outputs differ by summation only; a batch."""
+    import lit_llama.recurrence as R
+
+    r = np.random.RandomState(p)
+    B, T = 2, 200
+    proj = dev(r.randn(B * T, H * (2 * n + p)), torch.bfloat16)
+    decay = dev([0.0, 0.999, 0.7, 1.0][:H])
+    outs = []
+    for chunks in (True, False):
+        monkeypatch.setattr(R, "USE_CHUNKS", chunks)
+        state = torch.full((B, H, n, p), float("nan"), device="cuda")
+        y = R.decay_scan_constant(proj, 0, H * n, 2 * H * n, decay, True, 1.0, state, pos(0, T), B, T, H, H, n, p)
+        outs.append((host(y), host(state)))
+    close(outs[0][0], outs[1][0], 3e-5)
+    close(outs[0][1], outs[1][1], 2e-6)
+    act = rounded(O.silu(host(proj)[:T]), torch.bfloat16)
+    want = O.constant_decay_memory(act[:, :H * n].reshape(T, H, n), act[:, H * n:2 * H * n].reshape(T, H, n),
+                                   act[:, 2 * H * n:].reshape(T, H, p), host(decay)).reshape(T, -1)
+    close(outs[0][0][:T], want, 2e-3)                           # (a bf16 tie of the activation may round either way)
+
+
+def test_a_memory_read_back_across_many_chunks():
+    """Decay one: what a token wrote is read back 700 tokens and ten chunks later to fp32 accuracy, and nothing before it."""
+    import lit_llama.recurrence as R
+
+    T, n, p = 777, 16, 8
+    q, k, v = np.zeros((T, n)), np.zeros((T, n)), np.zeros((T, p))
+    k[65, 3], v[65] = 1.0, np.arange(1, p + 1)
+    q[64, 3], q[65, 3], q[66, 3], q[-1, 3] = 1.0, 1.0, 1.0, 1.0
+    state = torch.full((1, 1, n, p), float("nan"), device="cuda")
+    bfl = torch.bfloat16
+    y = host(R.decay_scan(dev(q, bfl), 0, dev(k, bfl), 0, dev(v, bfl), 0, dev(np.ones((T, 1))), False, None, None, 1.0, state, pos(0, T), 1, T,
+                          1, 1, n, p))
+    for t in (65, 66, T - 1):
+        close(y[t], np.arange(1, p + 1), 1e-6)
+    assert np.abs(y[:65]).max() == 0.0 and np.abs(y[67:-1]).max() == 0.0

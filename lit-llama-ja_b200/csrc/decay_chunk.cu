@@ -14,8 +14,9 @@
 
 namespace llb {
 
-constexpr int DC_L = 64, DC_PT = 64, DC_THREADS = 128;       // tokens of a chunk, value columns of a block
-constexpr int DC_LV = DC_PT + 8;
+// Blocks of eight warps: four rows of 16 x two halves of the block's PT value columns (64, or 128 for wide heads).  Everything a
+// block reads is requested before anything is worked on, so that a block waits for memory about once.
+constexpr int DC_L = 64, DC_THREADS = 256;                   // tokens of a chunk
 constexpr double DC_LOG_MIN = -1e4;                          // log of a decay of zero: e^-10000 is zero in fp32
 
 __device__ __forceinline__ void dc_ldmatrix(uint32_t (&r)[4], const void* p) {
@@ -65,39 +66,62 @@ __device__ __forceinline__ void dc_log_sums(const float* __restrict__ a, int a_r
   G[2 * lane + 1] = incl;
 }
 
+// Rows of a [64][cols] slice of an activation matrix (cols a multiple of 8, at most PAD), requested: unit it of a thread is 16 bytes.
+template <int PAD>
+struct DcTile {
+  static constexpr int UNITS = DC_L * (PAD / 8), IT = (UNITS + DC_THREADS - 1) / DC_THREADS;
+  uint4 u[IT];
+  __device__ __forceinline__ void load(const __nv_bfloat16* __restrict__ base, int stride, int len, int cols) {
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+      const int i = it * DC_THREADS + threadIdx.x, s = i / (PAD / 8), ch = (i % (PAD / 8)) * 8;
+      u[it] = make_uint4(0u, 0u, 0u, 0u);
+      if (i < UNITS && s < len && ch < cols) u[it] = *(const uint4*)(base + (size_t)s * stride + ch);
+    }
+  }
+  template <bool SILU>
+  __device__ __forceinline__ void store(__nv_bfloat16* smem, int ld) const {
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+      const int i = it * DC_THREADS + threadIdx.x, s = i / (PAD / 8), ch = (i % (PAD / 8)) * 8;
+      if (i < UNITS) *(uint4*)&smem[s * ld + ch] = dc_in8<SILU>(u[it]);
+    }
+  }
+};
+
 // grid (chunks * p tiles, H, B): D_c into dst[((b * H + h) * chunks + c)][n][p], e^(G_last) into total[(b * H + h) * chunks + c].
 // NP: n rounded up to 16, 32, 64 or 128.
-template <int NP, bool SILU>
-__global__ void __launch_bounds__(DC_THREADS) decay_collect_kernel(const __nv_bfloat16* __restrict__ k, int k_stride,
-                                                                   const __nv_bfloat16* __restrict__ v, int v_stride,
-                                                                   const float* __restrict__ a, int a_row, const float* __restrict__ ks,
-                                                                   float* __restrict__ dst, float* __restrict__ total, int Tn, int H,
-                                                                   int qk_heads, int n, int p, int ptiles) {
-  constexpr int LK = NP + 8;
+template <int NP, int PT, bool SILU>
+__global__ void __launch_bounds__(DC_THREADS, 2) decay_collect_kernel(const __nv_bfloat16* __restrict__ k, int k_stride,
+                                                                      const __nv_bfloat16* __restrict__ v, int v_stride,
+                                                                      const float* __restrict__ a, int a_row, const float* __restrict__ ks,
+                                                                      float* __restrict__ dst, float* __restrict__ total, int Tn, int H,
+                                                                      int qk_heads, int n, int p, int ptiles) {
+  constexpr int LK = NP + 8, LV = PT + 8, NF = PT / 16;        // NF: 8-column fragments of a warp's half
   extern __shared__ __align__(16) unsigned char dc_smem[];
   __nv_bfloat16* Ks = (__nv_bfloat16*)dc_smem;                // [3 terms][64][LK]
   __nv_bfloat16* Vs = Ks + 3 * DC_L * LK;                     // [64][LV]
   __shared__ double G[DC_L];
   __shared__ float wgt[DC_L];
-  const int c = blockIdx.x / ptiles, p0 = (blockIdx.x - c * ptiles) * DC_PT, h = blockIdx.y, b = blockIdx.z, g = h / (H / qk_heads);
+  const int c = blockIdx.x / ptiles, p0 = (blockIdx.x - c * ptiles) * PT, h = blockIdx.y, b = blockIdx.z, g = h / (H / qk_heads);
   const int chunks = gridDim.x / ptiles, t0 = c * DC_L, len = min(DC_L, Tn - t0), tid = threadIdx.x;
   const size_t m0 = (size_t)b * Tn + t0;
-  const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
+  DcTile<NP> kt;
+  DcTile<PT> vt;
+  kt.load(k + m0 * k_stride + (size_t)g * n, k_stride, len, n);
+  vt.load(v + m0 * v_stride + (size_t)h * p + p0, v_stride, len, p - p0);
+  const float ksv = (tid < len && ks) ? ks[(m0 + tid) * H + h] : 1.f;
   dc_log_sums(a, a_row, h, m0, len, G);
-  for (int i = tid; i < DC_L * (DC_PT / 8); i += DC_THREADS) {
-    const int s = i / (DC_PT / 8), ch = (i % (DC_PT / 8)) * 8;
-    uint4 u = zero4;
-    if (s < len && p0 + ch < p) u = dc_in8<SILU>(*(const uint4*)(v + (m0 + s) * v_stride + (size_t)h * p + p0 + ch));
-    *(uint4*)&Vs[s * DC_LV + ch] = u;
-  }
+  vt.template store<SILU>(Vs, LV);
   __syncthreads();
-  if (tid < DC_L) wgt[tid] = tid < len ? expf((float)(G[DC_L - 1] - G[tid])) * (ks ? ks[(m0 + tid) * H + h] : 1.f) : 0.f;
+  if (tid < DC_L) wgt[tid] = tid < len ? expf((float)(G[DC_L - 1] - G[tid])) * ksv : 0.f;
   if (tid == 0 && p0 == 0) total[((size_t)b * H + h) * chunks + c] = expf((float)G[DC_L - 1]);
   __syncthreads();
-  for (int i = tid; i < DC_L * (NP / 8); i += DC_THREADS) {
-    const int s = i / (NP / 8), ch = (i % (NP / 8)) * 8;
-    uint4 u = zero4;
-    if (s < len && ch < n) u = dc_in8<SILU>(*(const uint4*)(k + (m0 + s) * k_stride + (size_t)g * n + ch));
+#pragma unroll
+  for (int it = 0; it < DcTile<NP>::IT; ++it) {
+    const int i = it * DC_THREADS + tid, s = i / (NP / 8), ch = (i % (NP / 8)) * 8;
+    if (i >= DcTile<NP>::UNITS) break;
+    const uint4 u = dc_in8<SILU>(kt.u[it]);
     const float w = wgt[s];
     const uint32_t in[4] = {u.x, u.y, u.z, u.w};
     uint32_t out[3][4];
@@ -112,36 +136,36 @@ __global__ void __launch_bounds__(DC_THREADS) decay_collect_kernel(const __nv_bf
     for (int z = 0; z < 3; ++z) *(uint4*)&Ks[(z * DC_L + s) * LK + ch] = make_uint4(out[z][0], out[z][1], out[z][2], out[z][3]);
   }
   __syncthreads();
-  const int warp = tid >> 5, lane = tid & 31;
+  const int warp = tid >> 5, lane = tid & 31, c0 = (warp >> 2) * (PT / 2);
   float* D = dst + (((size_t)b * H + h) * chunks + c) * (size_t)n * p;
 #pragma unroll 1
-  for (int mt = warp; mt < NP / 16; mt += DC_THREADS / 32) {
+  for (int mt = warp & 3; mt < NP / 16; mt += 4) {
     if (mt * 16 >= n) break;
-    float acc[DC_PT / 8][4];
+    float acc[NF][4];
 #pragma unroll
-    for (int f = 0; f < DC_PT / 8; ++f) acc[f][0] = acc[f][1] = acc[f][2] = acc[f][3] = 0.f;
+    for (int f = 0; f < NF; ++f) acc[f][0] = acc[f][1] = acc[f][2] = acc[f][3] = 0.f;
 #pragma unroll
     for (int st = 0; st < DC_L / 16; ++st) {
-      uint32_t bf[DC_PT / 16][4];
+      uint32_t bf[NF / 2][4];
 #pragma unroll
-      for (int d = 0; d < DC_PT / 16; ++d)
-        dc_ldmatrix_trans(bf[d], &Vs[(st * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * DC_LV + d * 16 + (lane >> 4) * 8]);
+      for (int d = 0; d < NF / 2; ++d)
+        dc_ldmatrix_trans(bf[d], &Vs[(st * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LV + c0 + d * 16 + (lane >> 4) * 8]);
 #pragma unroll
       for (int z = 2; z >= 0; --z) {                          // the smallest term first
         uint32_t af[4];
         dc_ldmatrix_trans(af, &Ks[(z * DC_L + st * 16 + (lane & 7) + (lane >> 4) * 8) * LK + mt * 16 + ((lane >> 3) & 1) * 8]);
 #pragma unroll
-        for (int d = 0; d < DC_PT / 16; ++d) {
+        for (int d = 0; d < NF / 2; ++d) {
           mma_bf16_16816(acc[2 * d], af[0], af[1], af[2], af[3], bf[d][0], bf[d][1]);
           mma_bf16_16816(acc[2 * d + 1], af[0], af[1], af[2], af[3], bf[d][2], bf[d][3]);
         }
       }
     }
 #pragma unroll
-    for (int f = 0; f < DC_PT / 8; ++f)
+    for (int f = 0; f < NF; ++f)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const int i = mt * 16 + (lane >> 2) + e * 8, col = p0 + f * 8 + (lane & 3) * 2;
+        const int i = mt * 16 + (lane >> 2) + e * 8, col = p0 + c0 + f * 8 + (lane & 3) * 2;
         if (i < n && col < p) *(float2*)(D + (size_t)i * p + col) = make_float2(acc[f][2 * e], acc[f][2 * e + 1]);
       }
   }
@@ -176,55 +200,66 @@ __global__ void __launch_bounds__(128) decay_pass_kernel(float* __restrict__ chu
   *S = s;
 }
 
-// grid (chunks * p tiles, H, B).  A warp owns 16 consecutive tokens; its queries come from global memory straight into fragments.
-template <int NP, bool SILU>
-__global__ void __launch_bounds__(DC_THREADS, 3) decay_read_kernel(
+// grid (chunks * p tiles, H, B).  A warp owns 16 consecutive tokens and half of the block's columns; its queries come from global
+// memory straight into fragments.
+template <int NP, int PT, bool SILU>
+__global__ void __launch_bounds__(DC_THREADS, 2) decay_read_kernel(
     const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ k, int k_stride, const __nv_bfloat16* __restrict__ v,
     int v_stride, const float* __restrict__ a, int a_row, const float* __restrict__ ks, const float* __restrict__ skip, float qs,
     const float* __restrict__ chunk_state, const int32_t* __restrict__ pos_ids, float* __restrict__ y, int Tn, int H, int qk_heads, int n,
     int p, int ptiles) {
-  constexpr int LK = NP + 8;
+  constexpr int LK = NP + 8, LV = PT + 8, NF = PT / 16;
   extern __shared__ __align__(16) unsigned char dc_smem[];
   __nv_bfloat16* Ks = (__nv_bfloat16*)dc_smem;                // [64][LK]
   __nv_bfloat16* Vs = Ks + DC_L * LK;                         // [64][LV]
-  __nv_bfloat16* Ss = Vs + DC_L * DC_LV;                      // [2 terms][NP][LV]
+  __nv_bfloat16* Ss = Vs + DC_L * LV;                         // [2 terms][NP][LV]
   __shared__ double G[DC_L];
   __shared__ float kw[DC_L];
-  const int c = blockIdx.x / ptiles, p0 = (blockIdx.x - c * ptiles) * DC_PT, h = blockIdx.y, b = blockIdx.z, g = h / (H / qk_heads);
+  const int c = blockIdx.x / ptiles, p0 = (blockIdx.x - c * ptiles) * PT, h = blockIdx.y, b = blockIdx.z, g = h / (H / qk_heads);
   const int chunks = gridDim.x / ptiles, t0 = c * DC_L, len = min(DC_L, Tn - t0);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row0 = (warp & 3) * 16, c0 = (warp >> 2) * (PT / 2);
   const size_t m0 = (size_t)b * Tn + t0;
-  const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
   const bool has_state = c > 0 || pos_ids[0] != 0;
-  for (int i = tid; i < DC_L * (NP / 8); i += DC_THREADS) {
-    const int s = i / (NP / 8), ch = (i % (NP / 8)) * 8;
-    uint4 u = zero4;
-    if (s < len && ch < n) u = dc_in8<SILU>(*(const uint4*)(k + (m0 + s) * k_stride + (size_t)g * n + ch));
-    *(uint4*)&Ks[s * LK + ch] = u;
-  }
-  for (int i = tid; i < DC_L * (DC_PT / 8); i += DC_THREADS) {
-    const int s = i / (DC_PT / 8), ch = (i % (DC_PT / 8)) * 8;
-    uint4 u = zero4;
-    if (s < len && p0 + ch < p) u = dc_in8<SILU>(*(const uint4*)(v + (m0 + s) * v_stride + (size_t)h * p + p0 + ch));
-    *(uint4*)&Vs[s * DC_LV + ch] = u;
-  }
+  const float* S = chunk_state + (((size_t)b * H + h) * chunks + c) * (size_t)n * p;
+  DcTile<NP> kt;
+  DcTile<PT> vt;
+  kt.load(k + m0 * k_stride + (size_t)g * n, k_stride, len, n);
+  vt.load(v + m0 * v_stride + (size_t)h * p + p0, v_stride, len, p - p0);
+  const float ksv = (tid < len && ks) ? ks[(m0 + tid) * H + h] : 1.f;
+  // the state's rows in rounds of eight 16-byte units per thread: the first round is requested with the keys and values
+  constexpr int SU = NP * (PT / 4), SR = (SU + 8 * DC_THREADS - 1) / (8 * DC_THREADS);
+  float4 sv[8];
+  auto state_load = [&](int rd) {
+#pragma unroll
+    for (int it = 0; it < 8; ++it) {
+      const int i = (rd * 8 + it) * DC_THREADS + tid, r = i / (PT / 4), col = (i % (PT / 4)) * 4;
+      sv[it] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < SU && r < n && p0 + col < p) sv[it] = *(const float4*)(S + (size_t)r * p + p0 + col);
+    }
+  };
+  if (has_state) state_load(0);
+  kt.template store<SILU>(Ks, LK);
+  vt.template store<SILU>(Vs, LV);
   if (has_state) {
-    const float* S = chunk_state + (((size_t)b * H + h) * chunks + c) * (size_t)n * p;
-#pragma unroll 4
-    for (int i = tid; i < NP * (DC_PT / 4); i += DC_THREADS) {
-      const int r = i / (DC_PT / 4), col = (i % (DC_PT / 4)) * 4;
-      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (r < n && p0 + col < p) f = *(const float4*)(S + (size_t)r * p + p0 + col);
-      const uint32_t h0 = dc_term(f.x, f.y), h1 = dc_term(f.z, f.w);
-      *(uint2*)&Ss[r * DC_LV + col] = make_uint2(h0, h1);
-      *(uint2*)&Ss[(NP + r) * DC_LV + col] = make_uint2(dc_pack(f.x, f.y), dc_pack(f.z, f.w));
+#pragma unroll
+    for (int rd = 0; rd < SR; ++rd) {
+#pragma unroll
+      for (int it = 0; it < 8; ++it) {
+        const int i = (rd * 8 + it) * DC_THREADS + tid, r = i / (PT / 4), col = (i % (PT / 4)) * 4;
+        if (i >= SU) break;
+        float4 f = sv[it];
+        const uint32_t h0 = dc_term(f.x, f.y), h1 = dc_term(f.z, f.w);
+        *(uint2*)&Ss[r * LV + col] = make_uint2(h0, h1);
+        *(uint2*)&Ss[(NP + r) * LV + col] = make_uint2(dc_pack(f.x, f.y), dc_pack(f.z, f.w));
+      }
+      if (rd + 1 < SR) state_load(rd + 1);
     }
   }
-  if (tid < DC_L) kw[tid] = tid < len ? (ks ? ks[(m0 + tid) * H + h] : 1.f) * qs : 0.f;
+  if (tid < DC_L) kw[tid] = tid < len ? ksv * qs : 0.f;
   dc_log_sums(a, a_row, h, m0, len, G);
   // query fragments: rows (lane / 4) and + 8 of the warp's 16, columns (lane % 4) * 2 and + 8 of every 16
   uint32_t qf[NP / 16][4];
-  const int r0 = warp * 16 + (lane >> 2);
+  const int r0 = row0 + (lane >> 2);
 #pragma unroll
   for (int kk = 0; kk < NP / 16; ++kk)
 #pragma unroll
@@ -233,10 +268,10 @@ __global__ void __launch_bounds__(DC_THREADS, 3) decay_read_kernel(
       qf[kk][e] = (r < len && col < n) ? dc_in2<SILU>(*(const uint32_t*)(q + (m0 + r) * q_stride + (size_t)g * n + col)) : 0u;
     }
   __syncthreads();
-  if (warp * 16 >= len) return;
-  float o[DC_PT / 8][4];
+  if (row0 >= len) return;
+  float o[NF][4];
 #pragma unroll
-  for (int f = 0; f < DC_PT / 8; ++f) o[f][0] = o[f][1] = o[f][2] = o[f][3] = 0.f;
+  for (int f = 0; f < NF; ++f) o[f][0] = o[f][1] = o[f][2] = o[f][3] = 0.f;
   const double g0 = G[r0], g1 = G[r0 + 8];
   if (has_state) {
 #pragma unroll
@@ -244,19 +279,19 @@ __global__ void __launch_bounds__(DC_THREADS, 3) decay_read_kernel(
 #pragma unroll
       for (int z = 1; z >= 0; --z)
 #pragma unroll
-        for (int d = 0; d < DC_PT / 16; ++d) {
+        for (int d = 0; d < NF / 2; ++d) {
           uint32_t bf[4];
-          dc_ldmatrix_trans(bf, &Ss[(z * NP + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * DC_LV + d * 16 + (lane >> 4) * 8]);
+          dc_ldmatrix_trans(bf, &Ss[(z * NP + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LV + c0 + d * 16 + (lane >> 4) * 8]);
           mma_bf16_16816(o[2 * d], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], bf[0], bf[1]);
           mma_bf16_16816(o[2 * d + 1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], bf[2], bf[3]);
         }
     const float e0 = expf((float)g0) * qs, e1 = expf((float)g1) * qs;
 #pragma unroll
-    for (int f = 0; f < DC_PT / 8; ++f) o[f][0] *= e0, o[f][1] *= e0, o[f][2] *= e1, o[f][3] *= e1;
+    for (int f = 0; f < NF; ++f) o[f][0] *= e0, o[f][1] *= e0, o[f][2] *= e1, o[f][3] *= e1;
   }
 #pragma unroll
   for (int st = 0; st < DC_L / 16; ++st) {                    // 16 keys at a time, none that lie after all of the warp's tokens
-    if (st > warp) break;
+    if (st * 16 > row0) break;
     float sc[2][4];
 #pragma unroll
     for (int j = 0; j < 2; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
@@ -281,9 +316,9 @@ __global__ void __launch_bounds__(DC_THREADS, 3) decay_read_kernel(
       ah[2 * j + 1] = dc_term(sc[j][2], sc[j][3]), al[2 * j + 1] = dc_pack(sc[j][2], sc[j][3]);
     }
 #pragma unroll
-    for (int d = 0; d < DC_PT / 16; ++d) {
+    for (int d = 0; d < NF / 2; ++d) {
       uint32_t bf[4];
-      dc_ldmatrix_trans(bf, &Vs[(st * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * DC_LV + d * 16 + (lane >> 4) * 8]);
+      dc_ldmatrix_trans(bf, &Vs[(st * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * LV + c0 + d * 16 + (lane >> 4) * 8]);
       mma_bf16_16816(o[2 * d], al[0], al[1], al[2], al[3], bf[0], bf[1]);
       mma_bf16_16816(o[2 * d + 1], al[0], al[1], al[2], al[3], bf[2], bf[3]);
       mma_bf16_16816(o[2 * d], ah[0], ah[1], ah[2], ah[3], bf[0], bf[1]);
@@ -295,43 +330,43 @@ __global__ void __launch_bounds__(DC_THREADS, 3) decay_read_kernel(
   for (int e = 0; e < 2; ++e) {
     const int r = r0 + e * 8;
     if (r >= len) continue;
-    float* yr = y + (m0 + r) * (size_t)H * p + (size_t)h * p + p0;
+    float* yr = y + (m0 + r) * (size_t)H * p + (size_t)h * p + p0 + c0;
 #pragma unroll
-    for (int f = 0; f < DC_PT / 8; ++f) {
+    for (int f = 0; f < NF; ++f) {
       const int col = f * 8 + (lane & 3) * 2;
-      if (p0 + col >= p) continue;
+      if (p0 + c0 + col >= p) continue;
       float v0 = o[f][2 * e], v1 = o[f][2 * e + 1];
       if (skip) {
-        v0 += sk * __bfloat162float(Vs[r * DC_LV + col]);
-        v1 += sk * __bfloat162float(Vs[r * DC_LV + col + 1]);
+        v0 += sk * __bfloat162float(Vs[r * LV + c0 + col]);
+        v1 += sk * __bfloat162float(Vs[r * LV + c0 + col + 1]);
       }
       *(float2*)(yr + col) = make_float2(v0, v1);
     }
   }
 }
 
-template <int NP, bool SILU>
+template <int NP, int PT, bool SILU>
 static int decay_chunked_launch(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const float* a,
                                 int a_row, const float* ks, const float* skip, float qs, float* state, const int32_t* pos_ids, float* y,
                                 int B, int Tn, int H, int qk_heads, int n, int p, float* scratch, cudaStream_t st) {
-  const int chunks = (Tn + DC_L - 1) / DC_L, ptiles = (p + DC_PT - 1) / DC_PT, np4 = n * p / 4;
+  const int chunks = (Tn + DC_L - 1) / DC_L, ptiles = (p + PT - 1) / PT, np4 = n * p / 4;
   float* chunk_state = scratch;
   float* total = scratch + (size_t)B * H * chunks * n * p;
   const dim3 grid(chunks * ptiles, H, B);
-  constexpr int smem_c = (3 * DC_L * (NP + 8) + DC_L * DC_LV) * 2, smem_r = (DC_L * (NP + 8) + DC_L * DC_LV + 2 * NP * DC_LV) * 2;
+  constexpr int smem_c = (3 * DC_L * (NP + 8) + DC_L * (PT + 8)) * 2, smem_r = (DC_L * (NP + 8) + DC_L * (PT + 8) + 2 * NP * (PT + 8)) * 2;
   static bool sized = false;
   if (!sized) {
-    LL_CUDA(cudaFuncSetAttribute(decay_collect_kernel<NP, SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_c));
-    LL_CUDA(cudaFuncSetAttribute(decay_read_kernel<NP, SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_r));
+    LL_CUDA(cudaFuncSetAttribute(decay_collect_kernel<NP, PT, SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_c));
+    LL_CUDA(cudaFuncSetAttribute(decay_read_kernel<NP, PT, SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_r));
     sized = true;
   }
   typedef const __nv_bfloat16* in_t;
-  decay_collect_kernel<NP, SILU><<<grid, DC_THREADS, smem_c, st>>>((in_t)k, k_stride, (in_t)v, v_stride, a, a_row, ks, chunk_state, total, Tn, H,
+  decay_collect_kernel<NP, PT, SILU><<<grid, DC_THREADS, smem_c, st>>>((in_t)k, k_stride, (in_t)v, v_stride, a, a_row, ks, chunk_state, total, Tn, H,
                                                                   qk_heads, n, p, ptiles);
   LL_LAUNCH_OK("decay_collect_kernel");
   decay_pass_kernel<<<dim3((np4 + 127) / 128, B * H), 128, 0, st>>>(chunk_state, total, state, pos_ids, chunks, np4);
   LL_LAUNCH_OK("decay_pass_kernel");
-  decay_read_kernel<NP, SILU><<<grid, DC_THREADS, smem_r, st>>>((in_t)q, q_stride, (in_t)k, k_stride, (in_t)v, v_stride, a, a_row, ks, skip, qs,
+  decay_read_kernel<NP, PT, SILU><<<grid, DC_THREADS, smem_r, st>>>((in_t)q, q_stride, (in_t)k, k_stride, (in_t)v, v_stride, a, a_row, ks, skip, qs,
                                                                chunk_state, pos_ids, y, Tn, H, qk_heads, n, p, ptiles);
   LL_LAUNCH_OK("decay_read_kernel");
   return LL_OK;
@@ -366,8 +401,10 @@ int ll_decay_chunked(const void* q, int q_stride, const void* k, int k_stride, c
   cudaStream_t st = (cudaStream_t)stream;
   const int a_row = a_constant ? 0 : H;
 #define LL_DC_S(NP, SILU)                                                                                                              \
-  return decay_chunked_launch<NP, SILU>(q, q_stride, k, k_stride, v, v_stride, a, a_row, ks, skip, qs, state, pos_ids, y, B, T, H, qk_heads, \
-                                        n, p, scratch, st)
+  return p <= 64 ? decay_chunked_launch<NP, 64, SILU>(q, q_stride, k, k_stride, v, v_stride, a, a_row, ks, skip, qs, state, pos_ids, y, B, T, \
+                                                      H, qk_heads, n, p, scratch, st)                                                        \
+                 : decay_chunked_launch<NP, 128, SILU>(q, q_stride, k, k_stride, v, v_stride, a, a_row, ks, skip, qs, state, pos_ids, y, B, T, \
+                                                       H, qk_heads, n, p, scratch, st)
 #define LL_DC(NP)                  \
   if (n <= NP) {                   \
     if (act_silu) LL_DC_S(NP, true); \

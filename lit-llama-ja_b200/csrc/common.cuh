@@ -66,7 +66,13 @@ template <> struct dt<__half> {
 // rounding; the kernels that form it all do so here, so that they agree bit for bit.
 template <typename T> __device__ __forceinline__ float silu_act(float x);
 template <> __device__ __forceinline__ float silu_act<float>(float x) { return x / (1.f + expf(-x)); }
-template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float x) { return bf16r(__fdividef(x, 1.f + __expf(-x))); }
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+template <> __device__ __forceinline__ float silu_act<__nv_bfloat16>(float x) { return bf16r(silu_fast(x)); }
+// two numbers rounded to bf16 and packed, the first in the low half (one conversion instruction)
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

@@ -29,17 +29,16 @@ __device__ __forceinline__ void dc_ldmatrix_trans(uint32_t (&r)[4], const void* 
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
                : "r"(smem_u32(p)));
 }
-__device__ __forceinline__ uint32_t dc_pack(float a, float b) { return (uint32_t)f32_to_bf16_bits(a) | ((uint32_t)f32_to_bf16_bits(b) << 16); }
 // x as bf16 terms: the first of (a, b) packed, the rest left in a and b
 __device__ __forceinline__ uint32_t dc_term(float& a, float& b) {
-  const float ha = bf16r(a), hb = bf16r(b);
-  a -= ha, b -= hb;
-  return (uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(ha)) | ((uint32_t)__bfloat16_as_ushort(__float2bfloat16_rn(hb)) << 16);
+  const uint32_t u = pack_bf16(a, b);
+  a -= bf16_bits_to_f32(u & 0xffffu), b -= __uint_as_float(u & 0xffff0000u);
+  return u;
 }
 template <bool SILU>
 __device__ __forceinline__ uint32_t dc_in2(uint32_t u) {
   if (!SILU) return u;
-  return dc_pack(silu_act<__nv_bfloat16>(bf16_bits_to_f32(u & 0xffffu)), silu_act<__nv_bfloat16>(bf16_bits_to_f32(u >> 16)));
+  return pack_bf16(silu_fast(bf16_bits_to_f32(u & 0xffffu)), silu_fast(__uint_as_float(u & 0xffff0000u)));
 }
 template <bool SILU>
 __device__ __forceinline__ uint4 dc_in8(uint4 u) {
@@ -130,7 +129,7 @@ __global__ void __launch_bounds__(DC_THREADS, 2) decay_collect_kernel(const __nv
       float x0 = bf16_bits_to_f32(in[q] & 0xffffu) * w, x1 = bf16_bits_to_f32(in[q] >> 16) * w;
       out[0][q] = dc_term(x0, x1);
       out[1][q] = dc_term(x0, x1);
-      out[2][q] = dc_pack(x0, x1);
+      out[2][q] = pack_bf16(x0, x1);
     }
 #pragma unroll
     for (int z = 0; z < 3; ++z) *(uint4*)&Ks[(z * DC_L + s) * LK + ch] = make_uint4(out[z][0], out[z][1], out[z][2], out[z][3]);
@@ -171,30 +170,29 @@ __global__ void __launch_bounds__(DC_THREADS, 2) decay_collect_kernel(const __nv
   }
 }
 
-// Per (sequence, head), four neighbouring elements of the state a thread: D_c is replaced by the state before chunk c, the state
+// Per (sequence, head), two neighbouring elements of the state a thread: D_c is replaced by the state before chunk c, the state
 // after the last chunk goes back to `state`.
 __global__ void __launch_bounds__(128) decay_pass_kernel(float* __restrict__ chunk_state, const float* __restrict__ total,
                                                          float* __restrict__ state, const int32_t* __restrict__ pos_ids, int chunks,
-                                                         int np4) {
+                                                         int np2) {
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= np4) return;
+  if (i >= np2) return;
   const size_t bh = blockIdx.y;
-  float4* D = (float4*)chunk_state + bh * chunks * np4 + i;
-  float4* S = (float4*)state + bh * np4 + i;
+  float2* D = (float2*)chunk_state + bh * chunks * np2 + i;
+  float2* S = (float2*)state + bh * np2 + i;
   const float* tot = total + bh * chunks;
-  float4 s = pos_ids[0] == 0 ? make_float4(0.f, 0.f, 0.f, 0.f) : *S;
-  constexpr int AHEAD = 8;                                    // chunks whose loads are in flight together
+  float2 s = pos_ids[0] == 0 ? make_float2(0.f, 0.f) : *S;
+  constexpr int AHEAD = 16;                                   // chunks whose loads are in flight together
   for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-    float4 d[AHEAD];
-    float w[AHEAD];
+    float2 d[AHEAD];
 #pragma unroll
-    for (int j = 0; j < AHEAD; ++j)
-      if (c0 + j < chunks) d[j] = D[(size_t)(c0 + j) * np4], w[j] = tot[c0 + j];
+    for (int j = 0; j < AHEAD; ++j) d[j] = c0 + j < chunks ? D[(size_t)(c0 + j) * np2] : make_float2(0.f, 0.f);
 #pragma unroll
     for (int j = 0; j < AHEAD; ++j)
       if (c0 + j < chunks) {
-        D[(size_t)(c0 + j) * np4] = s;
-        s = make_float4(w[j] * s.x + d[j].x, w[j] * s.y + d[j].y, w[j] * s.z + d[j].z, w[j] * s.w + d[j].w);
+        const float w = tot[c0 + j];
+        D[(size_t)(c0 + j) * np2] = s;
+        s = make_float2(w * s.x + d[j].x, w * s.y + d[j].y);
       }
   }
   *S = s;
@@ -250,7 +248,7 @@ __global__ void __launch_bounds__(DC_THREADS, 2) decay_read_kernel(
         float4 f = sv[it];
         const uint32_t h0 = dc_term(f.x, f.y), h1 = dc_term(f.z, f.w);
         *(uint2*)&Ss[r * LV + col] = make_uint2(h0, h1);
-        *(uint2*)&Ss[(NP + r) * LV + col] = make_uint2(dc_pack(f.x, f.y), dc_pack(f.z, f.w));
+        *(uint2*)&Ss[(NP + r) * LV + col] = make_uint2(pack_bf16(f.x, f.y), pack_bf16(f.z, f.w));
       }
       if (rd + 1 < SR) state_load(rd + 1);
     }
@@ -312,8 +310,8 @@ __global__ void __launch_bounds__(DC_THREADS, 2) decay_read_kernel(
     uint32_t ah[4], al[4];
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
-      ah[2 * j] = dc_term(sc[j][0], sc[j][1]), al[2 * j] = dc_pack(sc[j][0], sc[j][1]);
-      ah[2 * j + 1] = dc_term(sc[j][2], sc[j][3]), al[2 * j + 1] = dc_pack(sc[j][2], sc[j][3]);
+      ah[2 * j] = dc_term(sc[j][0], sc[j][1]), al[2 * j] = pack_bf16(sc[j][0], sc[j][1]);
+      ah[2 * j + 1] = dc_term(sc[j][2], sc[j][3]), al[2 * j + 1] = pack_bf16(sc[j][2], sc[j][3]);
     }
 #pragma unroll
     for (int d = 0; d < NF / 2; ++d) {
@@ -349,7 +347,7 @@ template <int NP, int PT, bool SILU>
 static int decay_chunked_launch(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const float* a,
                                 int a_row, const float* ks, const float* skip, float qs, float* state, const int32_t* pos_ids, float* y,
                                 int B, int Tn, int H, int qk_heads, int n, int p, float* scratch, cudaStream_t st) {
-  const int chunks = (Tn + DC_L - 1) / DC_L, ptiles = (p + PT - 1) / PT, np4 = n * p / 4;
+  const int chunks = (Tn + DC_L - 1) / DC_L, ptiles = (p + PT - 1) / PT, np2 = n * p / 2;
   float* chunk_state = scratch;
   float* total = scratch + (size_t)B * H * chunks * n * p;
   const dim3 grid(chunks * ptiles, H, B);
@@ -364,7 +362,7 @@ static int decay_chunked_launch(const void* q, int q_stride, const void* k, int 
   decay_collect_kernel<NP, PT, SILU><<<grid, DC_THREADS, smem_c, st>>>((in_t)k, k_stride, (in_t)v, v_stride, a, a_row, ks, chunk_state, total, Tn, H,
                                                                   qk_heads, n, p, ptiles);
   LL_LAUNCH_OK("decay_collect_kernel");
-  decay_pass_kernel<<<dim3((np4 + 127) / 128, B * H), 128, 0, st>>>(chunk_state, total, state, pos_ids, chunks, np4);
+  decay_pass_kernel<<<dim3((np2 + 127) / 128, B * H), 128, 0, st>>>(chunk_state, total, state, pos_ids, chunks, np2);
   LL_LAUNCH_OK("decay_pass_kernel");
   decay_read_kernel<NP, PT, SILU><<<grid, DC_THREADS, smem_r, st>>>((in_t)q, q_stride, (in_t)k, k_stride, (in_t)v, v_stride, a, a_row, ks, skip, qs,
                                                                chunk_state, pos_ids, y, Tn, H, qk_heads, n, p, ptiles);

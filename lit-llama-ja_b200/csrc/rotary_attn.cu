@@ -98,7 +98,7 @@ __global__ void __launch_bounds__(QP_THREADS) qk_rotary_append_kernel(
 
 // Heads of a row normed one by one: a warp owns a head, its numbers pass through the warp's shared row (the rotation pairs
 // distant dimensions).  q heads, then k heads, then the values element by element over the whole block.
-constexpr int QH_WARPS = QP_THREADS / 32, QH_DIM = 256;
+constexpr int QH_MAX_WARPS = 16, QH_DIM = 256;
 
 template <typename T>
 __device__ __forceinline__ void qh_load2(const T* p, int i, int n, bool pair, float& a, float& b) {
@@ -130,25 +130,26 @@ __device__ __forceinline__ void qh_store2<__nv_bfloat16>(__nv_bfloat16* p, int i
   }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(QP_THREADS) qk_head_append_kernel(
+// R: runs of 64 dimensions a head spans
+template <typename T, int R>
+__global__ void __launch_bounds__(QH_MAX_WARPS * 32) qk_head_append_kernel(
     const T* __restrict__ q, int q_stride, const T* __restrict__ k, int k_stride, const T* __restrict__ v, int v_stride,
     const T* __restrict__ first, int first_stride, float lam, const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps,
     const float* __restrict__ freq, int rot_dims, float temp_coef, int temp_every, const int32_t* __restrict__ pos_ids,
     T* __restrict__ q_out, T* __restrict__ kc, T* __restrict__ vc, int Tn, int H, int G, int dim, int vdim, int ring, int pair) {
-  __shared__ float row[QH_WARPS][QH_DIM];
+  __shared__ float row[QH_MAX_WARPS][R * 64];
   const int m = blockIdx.x, b = m / Tn, t = m - b * Tn;
   const int p = pos_ids[t], warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = rot_dims >> 1;
   const float temp = temp_every > 0 ? 1.f + temp_coef * logf((float)((p + 1) / temp_every) + 1.f) : 1.f;
   const size_t slot = (size_t)b * ring + (size_t)(p % ring);
-  for (int hh = warp; hh < H + G; hh += QH_WARPS) {
+  for (int hh = warp; hh < H + G; hh += (int)(blockDim.x >> 5)) {
     const bool is_q = hh < H;
     const T* src = is_q ? q + (size_t)m * q_stride + (size_t)hh * dim : k + (size_t)m * k_stride + (size_t)(hh - H) * dim;
     T* dst = is_q ? q_out + ((size_t)m * H + hh) * dim : kc + (slot * G + (hh - H)) * dim;
     const float* nw = is_q ? q_norm : k_norm;
-    float e0[QH_DIM / 64], e1[QH_DIM / 64], ss = 0.f;
+    float e0[R], e1[R], ss = 0.f;
 #pragma unroll
-    for (int r = 0; r < QH_DIM / 64; ++r) {
+    for (int r = 0; r < R; ++r) {
       const int i = 2 * (lane + 32 * r);
       if (r * 64 < dim) {
         qh_load2<T>(src, i, dim, pair, e0[r], e1[r]);
@@ -160,7 +161,7 @@ __global__ void __launch_bounds__(QP_THREADS) qk_head_append_kernel(
     const float mult = is_q ? temp : 1.f;
     if (rot_dims > 0) __syncwarp();              // the row's readers of the head before are done
 #pragma unroll
-    for (int r = 0; r < QH_DIM / 64; ++r) {
+    for (int r = 0; r < R; ++r) {
       const int i = 2 * (lane + 32 * r);
       if (r * 64 < dim) {
         e0[r] *= kn, e1[r] *= kn;
@@ -178,7 +179,7 @@ __global__ void __launch_bounds__(QP_THREADS) qk_head_append_kernel(
     if (rot_dims > 0) {
       __syncwarp();
 #pragma unroll
-      for (int r = 0; r < QH_DIM / 64; ++r) {
+      for (int r = 0; r < R; ++r) {
         const int i = 2 * (lane + 32 * r);
         if (r * 64 < dim) {
 #pragma unroll
@@ -195,13 +196,13 @@ __global__ void __launch_bounds__(QP_THREADS) qk_head_append_kernel(
       }
     }
 #pragma unroll
-    for (int r = 0; r < QH_DIM / 64; ++r)
+    for (int r = 0; r < R; ++r)
       if (r * 64 < dim) qh_store2<T>(dst, 2 * (lane + 32 * r), dim, pair, e0[r], e1[r]);
   }
   T* vrow = vc + slot * (size_t)G * vdim;
   const T* vsrc = v + (size_t)m * v_stride;
   const T* fsrc = first ? first + (size_t)m * first_stride : nullptr;
-  for (int i = 2 * threadIdx.x; i < G * vdim; i += 2 * QP_THREADS) {
+  for (int i = 2 * threadIdx.x; i < G * vdim; i += 2 * blockDim.x) {
     float a, c;
     qh_load2<T>(vsrc, i, G * vdim, pair, a, c);
     if (fsrc) {
@@ -829,18 +830,26 @@ int ll_qk_head_append(const void* q, int q_stride, const void* k, int k_stride, 
   cudaStream_t st = (cudaStream_t)stream;
   const int pair = ((q_stride | k_stride | v_stride | (first ? first_stride : 0) | dim | vdim) & 1) == 0 &&
                    (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)first | (uintptr_t)q_out | (uintptr_t)kc | (uintptr_t)vc) & 3) == 0;
-#define LL_QH(T_)                                                                                                                     \
-  qk_head_append_kernel<T_><<<B * T, QP_THREADS, 0, st>>>((const T_*)q, q_stride, (const T_*)k, k_stride, (const T_*)v, v_stride,      \
+  const int threads = 32 * (H + G < QH_MAX_WARPS ? H + G : QH_MAX_WARPS);
+#define LL_QH_R(T_, R)                                                                                                                \
+  qk_head_append_kernel<T_, R><<<B * T, threads, 0, st>>>((const T_*)q, q_stride, (const T_*)k, k_stride, (const T_*)v, v_stride,      \
                                                           (const T_*)first, first_stride, lam, q_norm, k_norm, eps, freq, rot_dims,    \
                                                           temp_coef, temp_every, pos_ids, (T_*)q_out, (T_*)kc, (T_*)vc, T, H, G, dim,  \
                                                           vdim, ring, pair)
-  if (dtype == LL_F32) LL_QH(float);
-  else if (dtype == LL_BF16) LL_QH(__nv_bfloat16);
-  else {
+#define LL_QH(T_)                    \
+  if (dim <= 64) LL_QH_R(T_, 1);     \
+  else if (dim <= 128) LL_QH_R(T_, 2); \
+  else LL_QH_R(T_, 4)
+  if (dtype == LL_F32) {
+    LL_QH(float);
+  } else if (dtype == LL_BF16) {
+    LL_QH(__nv_bfloat16);
+  } else {
     set_error("qk_head_append: unsupported dtype %d", dtype);
     return LL_ERR_UNSUPPORTED;
   }
 #undef LL_QH
+#undef LL_QH_R
   LL_LAUNCH_OK("qk_head_append_kernel");
   return LL_OK;
 }

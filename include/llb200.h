@@ -22,7 +22,7 @@
 extern "C" {
 #endif
 
-#define LL_ABI_VERSION 16
+#define LL_ABI_VERSION 17
 
 #define LL_OK 0
 #define LL_ERR_ARG (-1)         /* bad shape / dtype / null pointer */
@@ -375,6 +375,9 @@ LL_API int ll_glu_clamp(const void* gu, int gu_stride, int ff, float limit, floa
  * shift 0: the plain silu-gated unit). */
 LL_API int ll_glu_unit(const void* gu, int gu_stride, int ff, float limit, float alpha, float shift, void* h, int dtype, int rows,
                        ll_stream stream);
+/* The same with a bias (fp32 [2 ff], added to [gate | up] before the clamps; NULL: none) and output rows h_stride apart. */
+LL_API int ll_glu_unit_rows(const void* gu, int gu_stride, int ff, const float* bias, float limit, float alpha, float shift, void* h,
+                            int h_stride, int dtype, int rows, ll_stream stream);
 
 /* ---------------------------------------------------------------------------------------
  * Latent attention over a ring cache of latent rows (csrc/latent_attn.cu).  A cache row is
@@ -401,6 +404,13 @@ LL_API int ll_latent_attn(const void* q_lat, long long qs_h, long long qs_m, con
                           const void* cache, void* out, long long os_h, long long os_m, int dtype, int B, int T, int n_head,
                           int kv_rank, int rot_dim, int rot_dims, int cache_len, int window, float scale, int splits,
                           float* scratch, ll_stream stream);
+/* The same with the number of bf16 terms the softmax weights enter the weighted sum with in the tensor-core form (1: rounded to
+ * bf16; 2: 16 bits of the fp32 weight). */
+LL_API int ll_latent_attn_terms(const void* q_lat, long long qs_h, long long qs_m, const void* proj, int proj_stride,
+                                int q_rot_col0, int q_head_stride, int gate_col0, const float* rope, const int32_t* pos_ids,
+                                const void* cache, void* out, long long os_h, long long os_m, int dtype, int B, int T, int n_head,
+                                int kv_rank, int rot_dim, int rot_dims, int cache_len, int window, float scale, int splits,
+                                int weight_terms, float* scratch, ll_stream stream);
 LL_API size_t ll_latent_attn_scratch_bytes(int M, int n_head, int kv_rank, int splits);
 
 /* ---------------------------------------------------------------------------------------
@@ -468,6 +478,10 @@ LL_API int ll_add_norm_pair(float* x, const void* a0, float s0, const void* a1, 
  * out = (x - mean) / sqrt(var + eps) * w + b, var the mean squared deviation (w, b fp32 [dim]; out in the activation dtype). */
 LL_API int ll_add_layer_norm(float* x, const void* a, float s, const float* w, const float* b, float eps, void* out, int act_dtype,
                              int rows, int dim, ll_stream stream);
+/* x[m][:] += s * (a + a_bias) + step, in place, fp32 (a: activation dtype, with its fp32 bias row; step: an fp32 row that joins every
+ * row of the stream; each optional); then, with out given, out = x / sqrt(mean(x^2) + eps) * w in the activation dtype. */
+LL_API int ll_add_rms_norm(float* x, const void* a, float s, const float* a_bias, const float* step, const float* w, float eps, void* out,
+                           int act_dtype, int rows, int dim, ll_stream stream);
 /* RMS norm of fp32 rows y in `groups` equal parts with a gate (activation dtype, row stride gate_stride; silu, or a sigmoid
  * when gate_sigmoid):  gate_first 1: (y * gate(g)) / rms_part(.) * w;  0: y / rms_part(y) * w * gate(g).  w: C entries, or
  * C / groups shared by the parts (w_shared).  A part of y spans y_gs numbers (0: C / groups), of which the first C / groups are
@@ -476,6 +490,10 @@ LL_API int ll_add_layer_norm(float* x, const void* a, float s, const float* w, c
 LL_API int ll_gated_group_norm(const float* y, int y_gs, const float* stab, const void* gate, int gate_stride, const float* w,
                                int w_shared, float eps, int groups, int gate_first, int gate_sigmoid, void* out, int act_dtype,
                                int rows, int C, ll_stream stream);
+/* The same with output rows out_stride apart. */
+LL_API int ll_gated_group_norm_rows(const float* y, int y_gs, const float* stab, const void* gate, int gate_stride, const float* w,
+                                    int w_shared, float eps, int groups, int gate_first, int gate_sigmoid, void* out, int out_stride,
+                                    int act_dtype, int rows, int C, ll_stream stream);
 /* h <- relu(h)^2, in place */
 LL_API int ll_relu_squared(void* h, int dtype, size_t n, ll_stream stream);
 /* h <- gelu(h), in place: 0.5 h (1 + erf(h / sqrt 2)), or with tanh_form 0.5 h (1 + tanh(sqrt(2/pi) (h + 0.044715 h^3))) */
@@ -538,6 +556,25 @@ LL_API int ll_decay_chunked(const void* q, int q_stride, const void* k, int k_st
                             const float* a, int a_constant, int act_silu, const float* ks, const float* skip, float qs, float* state,
                             const int32_t* pos_ids, float* y, int B, int T, int H, int qk_heads, int n, int p, float* scratch,
                             ll_stream stream);
+/* Gated delta rule (csrc/delta_rule.cu), per sequence b and head h with S an n x p matrix, q and k of head h / (H / qk_heads):
+ *   k^ = k / sqrt(|k|^2 + unit_eps),  q^ = q / sqrt(|q|^2 + unit_eps) * qs
+ *   g = exp(-exp(a_log[h]) * softplus(raw_a + dt_bias[h])),  beta = sigmoid(raw_b)
+ *   S <- g S;  S <- S + k^ (beta (v - S^T k^))^T;  y = S^T q^
+ * q, k, v, raw_a, raw_b: column slices in the activation dtype (row strides given); state fp32 [B][H][n][p], advanced in place (zero
+ * before a sequence whose pos_ids[0] == 0); y fp32 [B*T][H*p].  n up to 512. */
+LL_API int ll_delta_scan(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const void* raw_a,
+                         const void* raw_b, int gate_stride, int dtype, const float* dt_bias, const float* a_log, float unit_eps,
+                         float qs, float* state, const int32_t* pos_ids, float* y, int B, int T, int H, int qk_heads, int n, int p,
+                         ll_stream stream);
+/* The same for bf16 prompts in chunks of 64 tokens on tensor cores (csrc/delta_chunk.cu).  ll_delta_chunked_supported: bf16,
+ * T >= 64, n <= 128 and p in multiples of 8, strides too; q, k, v, state, y and scratch (ll_delta_chunked_scratch_bytes) on 16-byte
+ * boundaries. */
+LL_API int ll_delta_chunked_supported(int dtype, int T, int n, int p, int q_stride, int k_stride, int v_stride);
+LL_API size_t ll_delta_chunked_scratch_bytes(int B, int T, int H, int n, int p);
+LL_API int ll_delta_chunked(const void* q, int q_stride, const void* k, int k_stride, const void* v, int v_stride, const void* raw_a,
+                            const void* raw_b, int gate_stride, int dtype, const float* dt_bias, const float* a_log, float unit_eps,
+                            float qs, float* state, const int32_t* pos_ids, float* y, int B, int T, int H, int qk_heads, int n, int p,
+                            float* scratch, ll_stream stream);
 /* Exponential gates with a running stabiliser, per (b, h): li = cap(raw_i + bias_i[h]), lf = logsigmoid(cap(raw_f + bias_f[h])),
  * cap(z) = c tanh(z / c) (c <= 0: none); mx_t = max(lf_t + mx_(t-1), li_t) with mx carried in mstate fp32 [B][H] (0 when
  * pos_ids[0] == 0); keep = exp(lf + mx_(t-1) - mx_t), take = exp(li - mx_t), stab = mx_t   (fp32 [B*T][H] each). */
@@ -619,6 +656,12 @@ LL_API int ll_softmax_attn_biased(const void* q, int q_stride, const void* gate,
                                   float softcap, int B, int T, int H, int G, int dim, int vdim, int window, int chunk, int ring,
                                   int splits, int form, int maps, float diff_lambda, float diff_post, float eps, float* scratch,
                                   void* y, ll_stream stream);
+/* The same with output rows y_stride (>= H * vdim) apart. */
+LL_API int ll_softmax_attn_rows(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc,
+                                int dtype, const int32_t* pos_ids, const float* sink, const float* slopes, float scale,
+                                float softcap, int B, int T, int H, int G, int dim, int vdim, int window, int chunk, int ring,
+                                int splits, int form, int maps, float diff_lambda, float diff_post, float eps, float* scratch,
+                                void* y, int y_stride, ll_stream stream);
 
 #ifdef __cplusplus
 }

@@ -25,6 +25,7 @@ FAMILY_SOURCES = {
     "Bededra": ["quant_pack", "residual_ops", "short_conv", "decay_scan", "decay_chunk", "window_attn", "moe_ops", "moe_gemm_tc"],
     "Tebodra": ["quant_pack", "residual_ops", "short_conv", "decay_scan", "rotary_attn"],
     "Livasun": ["quant_pack", "residual_ops", "short_conv", "decay_scan", "decay_chunk", "rotary_attn", "moe_ops", "moe_gemm_tc"],
+    "Zekonex": ["quant_pack", "residual_ops", "short_conv", "delta_rule", "delta_chunk", "rotary_attn", "latent_attn"],
     "Bumulix": ["quant_pack", "residual_ops", "rotary_attn", "latent_attn"],
 }
 

@@ -10,40 +10,12 @@
 // e^(..) ks k enters D as three bf16 terms (24 bits: what is carried on is as exact as the walk's fp32), the chunk's weights and
 // the state meet v and q as two terms (16 bits, the sum of both products in fp32).  Sums of log a are formed in fp64, so that the
 // difference of two of them keeps its digits whatever lies before it in the chunk.  The state handed on is fp32.
-#include "common.cuh"
+#include "chunk_mma.cuh"
 
 namespace llb {
 
 // Blocks of eight warps: four rows of 16 x two halves of the block's PT value columns (64, or 128 for wide heads).  Everything a
 // block reads is requested before anything is worked on, so that a block waits for memory about once.
-constexpr int DC_L = 64, DC_THREADS = 256;                   // tokens of a chunk
-constexpr double DC_LOG_MIN = -1e4;                          // log of a decay of zero: e^-10000 is zero in fp32
-
-__device__ __forceinline__ void dc_ldmatrix(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(smem_u32(p)));
-}
-__device__ __forceinline__ void dc_ldmatrix_trans(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-               : "r"(smem_u32(p)));
-}
-// x as bf16 terms: the first of (a, b) packed, the rest left in a and b
-__device__ __forceinline__ uint32_t dc_term(float& a, float& b) {
-  const uint32_t u = pack_bf16(a, b);
-  a -= bf16_bits_to_f32(u & 0xffffu), b -= __uint_as_float(u & 0xffff0000u);
-  return u;
-}
-template <bool SILU>
-__device__ __forceinline__ uint32_t dc_in2(uint32_t u) {
-  if (!SILU) return u;
-  return pack_bf16(silu_fast(bf16_bits_to_f32(u & 0xffffu)), silu_fast(__uint_as_float(u & 0xffff0000u)));
-}
-template <bool SILU>
-__device__ __forceinline__ uint4 dc_in8(uint4 u) {
-  return make_uint4(dc_in2<SILU>(u.x), dc_in2<SILU>(u.y), dc_in2<SILU>(u.z), dc_in2<SILU>(u.w));
-}
 
 // G[t] = sum over the chunk's tokens up to t of log a (tokens past the end: a = 1), by the first warp, two tokens a lane
 __device__ __forceinline__ void dc_log_sums(const float* __restrict__ a, int a_row, int h, size_t m0, int len, double* G) {
@@ -55,38 +27,8 @@ __device__ __forceinline__ void dc_log_sums(const float* __restrict__ a, int a_r
     const int t = 2 * lane + e;
     v[e] = t < len ? fmax((double)logf(a[(m0 + t) * a_row + h]), DC_LOG_MIN) : 0.0;
   }
-  double incl = v[0] + v[1];
-#pragma unroll
-  for (int d = 1; d < 32; d <<= 1) {
-    const double o = __shfl_up_sync(0xffffffffu, incl, d);
-    if (lane >= d) incl += o;
-  }
-  G[2 * lane] = incl - v[1];
-  G[2 * lane + 1] = incl;
+  dc_running_sums(v, G);
 }
-
-// Rows of a [64][cols] slice of an activation matrix (cols a multiple of 8, at most PAD), requested: unit it of a thread is 16 bytes.
-template <int PAD>
-struct DcTile {
-  static constexpr int UNITS = DC_L * (PAD / 8), IT = (UNITS + DC_THREADS - 1) / DC_THREADS;
-  uint4 u[IT];
-  __device__ __forceinline__ void load(const __nv_bfloat16* __restrict__ base, int stride, int len, int cols) {
-#pragma unroll
-    for (int it = 0; it < IT; ++it) {
-      const int i = it * DC_THREADS + threadIdx.x, s = i / (PAD / 8), ch = (i % (PAD / 8)) * 8;
-      u[it] = make_uint4(0u, 0u, 0u, 0u);
-      if (i < UNITS && s < len && ch < cols) u[it] = *(const uint4*)(base + (size_t)s * stride + ch);
-    }
-  }
-  template <bool SILU>
-  __device__ __forceinline__ void store(__nv_bfloat16* smem, int ld) const {
-#pragma unroll
-    for (int it = 0; it < IT; ++it) {
-      const int i = it * DC_THREADS + threadIdx.x, s = i / (PAD / 8), ch = (i % (PAD / 8)) * 8;
-      if (i < UNITS) *(uint4*)&smem[s * ld + ch] = dc_in8<SILU>(u[it]);
-    }
-  }
-};
 
 // grid (chunks * p tiles, H, B): D_c into dst[((b * H + h) * chunks + c)][n][p], e^(G_last) into total[(b * H + h) * chunks + c].
 // NP: n rounded up to 16, 32, 64 or 128.

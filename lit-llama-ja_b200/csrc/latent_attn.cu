@@ -210,7 +210,8 @@ __global__ void __launch_bounds__(LA_THREADS) latent_attn_kernel(const LatentAtt
 // A block owns 32 query rows = (a few consecutive tokens) x (up to 32 heads) and walks the union of their windows in
 // chunks of 64 cache rows: S = Q K^T (all heads against the same rows; a warp takes 16 rows x 16 keys x half of the row's
 // dimensions, the two halves meet in shared memory), online softmax in fp32, O += P C with the accumulators of the
-// 32 x kv_rank output split by columns over the 16 warps (NTW n-tiles of 8 columns each).  Sixteen warps, four per
+// 32 x kv_rank output split by columns over the 16 warps (NTW n-tiles of 8 columns each).  The weights P enter that product
+// rounded to bf16, or (TERMS = 2) as two bf16 terms whose sum carries 16 bits of the fp32 weight.  Sixteen warps, four per
 // scheduler: every phase is a chain of shared-memory loads and tensor instructions whose latency the other warps cover.
 constexpr int LM_ROWS = 32, LM_KC = 64;
 
@@ -236,7 +237,7 @@ struct LatentMmaGeom {
 
 // WARPS = 16: one block per SM, four warps per scheduler, the score product split over halves of the dimensions.
 // WARPS = 8: for rows short enough that two blocks share an SM (the same number of warps, two chunks in different phases).
-template <int NTW, int WARPS>
+template <int NTW, int WARPS, int TERMS>
 __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) latent_attn_mma_kernel(const LatentAttnParams P, const LatentMmaGeom G) {
   constexpr int LM_THREADS = WARPS * 32, LM_WARPS = WARPS;
   extern __shared__ __align__(16) unsigned char la_smem[];
@@ -244,8 +245,9 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) latent_attn_mm
   const int pitch = G.pitch;
   __nv_bfloat16* Qs = (__nv_bfloat16*)la_smem;                 // [32][pitch]
   __nv_bfloat16* Ks0 = Qs + LM_ROWS * pitch;                   // [2 stages][64][pitch]
-  __nv_bfloat16* Ps = Ks0 + 2 * LM_KC * pitch;                 // [32][64 + 8]
-  float* Ss = (float*)(Ps + LM_ROWS * (LM_KC + 8));            // [2 halves of the row's dimensions][32][64 + 1]
+  constexpr int PS = LM_ROWS * (LM_KC + 8);                    // one term of the weights
+  __nv_bfloat16* Ps = Ks0 + 2 * LM_KC * pitch;                 // [TERMS][32][64 + 8]
+  float* Ss = (float*)(Ps + TERMS * PS);                       // [2 halves of the row's dimensions][32][64 + 1]
   float* m_run = Ss + (WARPS == 16 ? 2 : 1) * LM_ROWS * (LM_KC + 1);   // [32]
   float* l_run = m_run + LM_ROWS;
   float* corr = l_run + LM_ROWS;
@@ -417,7 +419,14 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) latent_attn_mm
       const __nv_bfloat16 b0 = __float2bfloat16_rn(p0), b1 = __float2bfloat16_rn(p1);
       Ps[r * (LM_KC + 8) + lane] = b0;
       Ps[r * (LM_KC + 8) + lane + 32] = b1;
-      const float sum = warp_sum(__bfloat162float(b0) + __bfloat162float(b1));   // the weights as the product below sees them
+      float w0 = __bfloat162float(b0), w1 = __bfloat162float(b1);
+      if constexpr (TERMS == 2) {
+        const __nv_bfloat16 d0 = __float2bfloat16_rn(p0 - w0), d1 = __float2bfloat16_rn(p1 - w1);
+        Ps[PS + r * (LM_KC + 8) + lane] = d0;
+        Ps[PS + r * (LM_KC + 8) + lane + 32] = d1;
+        w0 += __bfloat162float(d0), w1 += __bfloat162float(d1);
+      }
+      const float sum = warp_sum(w0 + w1);       // the weights as the product below sees them
       if (lane == 0) {
         const float c = (mo == -INFINITY) ? 0.f : expf(mo - mn);
         corr[r] = c;
@@ -435,14 +444,15 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) latent_attn_mm
       }
 #pragma unroll
       for (int ks = 0; ks < LM_KC / 16; ++ks) {
-        uint32_t af[2][4];
+        uint32_t af[2 * TERMS][4];               // row tile i, term z at z * 2 + i
 #pragma unroll
-        for (int i = 0; i < 2; ++i) la_ldmatrix_x4(af[i], Ps + (i * 16 + (lane & 15)) * (LM_KC + 8) + ks * 16 + (lane >> 4) * 8);
+        for (int i = 0; i < 2 * TERMS; ++i)
+          la_ldmatrix_x4(af[i], Ps + (i >> 1) * PS + ((i & 1) * 16 + (lane & 15)) * (LM_KC + 8) + ks * 16 + (lane >> 4) * 8);
         if (NTW == 1) {
           uint32_t bf[2];
           la_ldmatrix_x2_trans(bf, Ks + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + wcol0);
 #pragma unroll
-          for (int i = 0; i < 2; ++i) mma_bf16_16816(acc[i][0], af[i][0], af[i][1], af[i][2], af[i][3], bf[0], bf[1]);
+          for (int i = 2 * TERMS - 1; i >= 0; --i) mma_bf16_16816(acc[i & 1][0], af[i][0], af[i][1], af[i][2], af[i][3], bf[0], bf[1]);
         } else {
 #pragma unroll
           for (int jp = 0; jp < NTW / 2; ++jp) {
@@ -450,9 +460,9 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) latent_attn_mm
             uint32_t bf[4];
             la_ldmatrix_x4_trans(bf, Ks + (ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + wcol0 + jp * 16 + (lane >> 4) * 8);
 #pragma unroll
-            for (int i = 0; i < 2; ++i) {
-              mma_bf16_16816(acc[i][2 * jp], af[i][0], af[i][1], af[i][2], af[i][3], bf[0], bf[1]);
-              mma_bf16_16816(acc[i][2 * jp + 1], af[i][0], af[i][1], af[i][2], af[i][3], bf[2], bf[3]);
+            for (int i = 2 * TERMS - 1; i >= 0; --i) {
+              mma_bf16_16816(acc[i & 1][2 * jp], af[i][0], af[i][1], af[i][2], af[i][3], bf[0], bf[1]);
+              mma_bf16_16816(acc[i & 1][2 * jp + 1], af[i][0], af[i][1], af[i][2], af[i][3], bf[2], bf[3]);
             }
           }
         }
@@ -499,21 +509,21 @@ __global__ void __launch_bounds__(WARPS * 32, WARPS == 8 ? 2 : 1) latent_attn_mm
   }
 }
 
-static size_t latent_mma_smem(int pitch, int halves) {
-  return sizeof(__nv_bfloat16) * ((size_t)(LM_ROWS + 2 * LM_KC) * pitch + (size_t)LM_ROWS * (LM_KC + 8)) +
+static size_t latent_mma_smem(int pitch, int halves, int terms) {
+  return sizeof(__nv_bfloat16) * ((size_t)(LM_ROWS + 2 * LM_KC) * pitch + (size_t)terms * LM_ROWS * (LM_KC + 8)) +
          sizeof(float) * ((size_t)halves * LM_ROWS * (LM_KC + 1) + 3 * LM_ROWS) + sizeof(int) * LM_ROWS;
 }
 
-template <int NTW, int WARPS>
+template <int NTW, int WARPS, int TERMS>
 static int launch_latent_mma(const LatentAttnParams& P, const LatentMmaGeom& G, int B, cudaStream_t st) {
-  const size_t smem = latent_mma_smem(G.pitch, WARPS == 16 ? 2 : 1);
+  const size_t smem = latent_mma_smem(G.pitch, WARPS == 16 ? 2 : 1, TERMS);
   static size_t configured = 0;
   if (smem > configured) {
-    LL_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<NTW, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    LL_CUDA(cudaFuncSetAttribute(latent_attn_mma_kernel<NTW, WARPS, TERMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     configured = smem;
   }
   dim3 grid(B * ((P.Tn + G.TQ - 1) / G.TQ), (P.H + G.HB - 1) / G.HB, P.splits);
-  latent_attn_mma_kernel<NTW, WARPS><<<grid, WARPS * 32, smem, st>>>(P, G);
+  latent_attn_mma_kernel<NTW, WARPS, TERMS><<<grid, WARPS * 32, smem, st>>>(P, G);
   LL_LAUNCH_OK("latent_attn_mma_kernel");
   return LL_OK;
 }
@@ -605,9 +615,17 @@ int ll_latent_attn(const void* q_lat, long long qs_h, long long qs_m, const void
                    int q_head_stride, int gate_col0, const float* rope, const int32_t* pos_ids, const void* cache, void* out,
                    long long os_h, long long os_m, int dtype, int B, int T, int n_head, int kv_rank, int rot_dim, int rot_dims,
                    int cache_len, int window, float scale, int splits, float* scratch, ll_stream stream) {
+  return ll_latent_attn_terms(q_lat, qs_h, qs_m, proj, proj_stride, q_rot_col0, q_head_stride, gate_col0, rope, pos_ids, cache, out, os_h,
+                              os_m, dtype, B, T, n_head, kv_rank, rot_dim, rot_dims, cache_len, window, scale, splits, 1, scratch, stream);
+}
+
+int ll_latent_attn_terms(const void* q_lat, long long qs_h, long long qs_m, const void* proj, int proj_stride, int q_rot_col0,
+                         int q_head_stride, int gate_col0, const float* rope, const int32_t* pos_ids, const void* cache, void* out,
+                         long long os_h, long long os_m, int dtype, int B, int T, int n_head, int kv_rank, int rot_dim, int rot_dims,
+                         int cache_len, int window, float scale, int splits, int weight_terms, float* scratch, ll_stream stream) {
   LL_CHECK_ARG(q_lat && proj && rope && pos_ids && cache && out, "latent_attn: null pointer");
   LL_CHECK_ARG(B >= 0 && T >= 0 && n_head > 0 && kv_rank > 0 && rot_dim >= 0 && rot_dims >= 0 && rot_dims <= rot_dim &&
-                   rot_dims % 2 == 0 && cache_len > 0 && splits >= 1 && (splits == 1 || scratch),
+                   rot_dims % 2 == 0 && cache_len > 0 && splits >= 1 && (splits == 1 || scratch) && (weight_terms == 1 || weight_terms == 2),
                "bad latent_attn arguments");
   if (B * T == 0) return LL_OK;
   if (kv_rank > LA_THREADS * LA_NACC) {
@@ -636,21 +654,23 @@ int ll_latent_attn(const void* q_lat, long long qs_h, long long qs_m, const void
     if (G.TQ < 1) G.TQ = 1;
     G.DKP = (Dk + 15) / 16 * 16;
     G.pitch = G.DKP + 8;
-    if (latent_mma_smem(G.pitch, 2) <= 220 * 1024) {
+    if (latent_mma_smem(G.pitch, 2, weight_terms) <= 220 * 1024) {
       // two 8-warp blocks per SM when two fit (shared memory, and 32 columns of O per warp at most), else one of 16 warps
-      const bool pair = 2 * (latent_mma_smem(G.pitch, 1) + 1024) <= 227 * 1024 && kv_rank <= 256;
+      const bool pair = 2 * (latent_mma_smem(G.pitch, 1, weight_terms) + 1024) <= 227 * 1024 && kv_rank <= 256;
       const int warps = pair ? 8 : 16;
       const int cols_per_warp = (kv_rank + warps - 1) / warps;
       int rc;
+#define LL_LM(NTW, WARPS) (weight_terms == 2 ? launch_latent_mma<NTW, WARPS, 2>(P, G, B, st) : launch_latent_mma<NTW, WARPS, 1>(P, G, B, st))
       if (pair) {
-        if (cols_per_warp <= 8) rc = launch_latent_mma<1, 8>(P, G, B, st);
-        else if (cols_per_warp <= 16) rc = launch_latent_mma<2, 8>(P, G, B, st);
-        else rc = launch_latent_mma<4, 8>(P, G, B, st);
+        if (cols_per_warp <= 8) rc = LL_LM(1, 8);
+        else if (cols_per_warp <= 16) rc = LL_LM(2, 8);
+        else rc = LL_LM(4, 8);
       } else {
-        if (cols_per_warp <= 8) rc = launch_latent_mma<1, 16>(P, G, B, st);
-        else if (cols_per_warp <= 16) rc = launch_latent_mma<2, 16>(P, G, B, st);
-        else rc = launch_latent_mma<4, 16>(P, G, B, st);
+        if (cols_per_warp <= 8) rc = LL_LM(1, 16);
+        else if (cols_per_warp <= 16) rc = LL_LM(2, 16);
+        else rc = LL_LM(4, 16);
       }
+#undef LL_LM
       if (rc != LL_OK) return rc;
       done = true;
     }

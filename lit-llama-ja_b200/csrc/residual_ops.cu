@@ -103,19 +103,22 @@ __device__ __forceinline__ float glu_unit(float g, float u, float limit, float a
   u = fminf(fmaxf(u, -limit), limit);
   return g / (1.f + expf(-alpha * g)) * (u + shift);
 }
+// bias (optional): fp32 [2 ff], added to [gate | up] before the clamps; rows of h lie h_stride apart
 template <typename T>
-__global__ void glu_unit_kernel(const T* __restrict__ gu, int gu_stride, int ff, float limit, float alpha, float shift,
-                                T* __restrict__ h, size_t n) {
+__global__ void glu_unit_kernel(const T* __restrict__ gu, int gu_stride, int ff, const float* __restrict__ bias, float limit, float alpha,
+                                float shift, T* __restrict__ h, int h_stride, size_t n) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n) return;
   const size_t m = i / ff;
   const int c = (int)(i - m * ff);
-  dt<T>::st(h, i, glu_unit(dt<T>::ld(gu, m * gu_stride + c), dt<T>::ld(gu, m * gu_stride + ff + c), limit, alpha, shift));
+  float g = dt<T>::ld(gu, m * gu_stride + c), u = dt<T>::ld(gu, m * gu_stride + ff + c);
+  if (bias) g += bias[c], u += bias[ff + c];
+  dt<T>::st(h, m * h_stride + c, glu_unit(g, u, limit, alpha, shift));
 }
 // ff, gu_stride multiples of 8 and 16-byte aligned rows: a thread owns eight columns of one row
 template <typename T>
-__global__ void glu_unit8_kernel(const T* __restrict__ gu, int gu_stride, int ff, float limit, float alpha, float shift,
-                                 T* __restrict__ h, int n8) {
+__global__ void glu_unit8_kernel(const T* __restrict__ gu, int gu_stride, int ff, const float* __restrict__ bias, float limit, float alpha,
+                                 float shift, T* __restrict__ h, int h_stride, int n8) {
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n8) return;
   const int per = ff / 8, m = i / per, c = (i - m * per) * 8;
@@ -123,20 +126,29 @@ __global__ void glu_unit8_kernel(const T* __restrict__ gu, int gu_stride, int ff
   float g[8], u[8];
   ld8<T>(row, g);
   ld8<T>(row + ff, u);
+  if (bias) {
+    float bg[8], bu[8];
+    ld8<float>(bias + c, bg);
+    ld8<float>(bias + ff + c, bu);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) g[e] += bg[e], u[e] += bu[e];
+  }
 #pragma unroll
   for (int e = 0; e < 8; ++e) g[e] = glu_unit(g[e], u[e], limit, alpha, shift);
-  st8<T>(h + (size_t)m * ff + c, g);
+  st8<T>(h + (size_t)m * h_stride + c, g);
 }
 
 template <typename T>
-static int glu_unit_launch(const void* gu, int gu_stride, int ff, float limit, float alpha, float shift, void* h, int rows,
-                           cudaStream_t st) {
+static int glu_unit_launch(const void* gu, int gu_stride, int ff, const float* bias, float limit, float alpha, float shift, void* h,
+                           int h_stride, int rows, cudaStream_t st) {
   const size_t n = (size_t)rows * ff;
-  if (ff % 8 == 0 && gu_stride % 8 == 0 && (((uintptr_t)gu | (uintptr_t)h) & 15) == 0 && n / 8 < (1ull << 31)) {
+  if (ff % 8 == 0 && gu_stride % 8 == 0 && h_stride % 8 == 0 && (((uintptr_t)gu | (uintptr_t)h | (uintptr_t)bias) & 15) == 0 &&
+      n / 8 < (1ull << 31)) {
     const int n8 = (int)(n / 8);
-    glu_unit8_kernel<T><<<(n8 + 127) / 128, 128, 0, st>>>((const T*)gu, gu_stride, ff, limit, alpha, shift, (T*)h, n8);
+    glu_unit8_kernel<T><<<(n8 + 127) / 128, 128, 0, st>>>((const T*)gu, gu_stride, ff, bias, limit, alpha, shift, (T*)h, h_stride, n8);
   } else {
-    glu_unit_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, st>>>((const T*)gu, gu_stride, ff, limit, alpha, shift, (T*)h, n);
+    glu_unit_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, st>>>((const T*)gu, gu_stride, ff, bias, limit, alpha, shift, (T*)h, h_stride,
+                                                                    n);
   }
   LL_LAUNCH_OK("glu_unit_kernel");
   return LL_OK;
@@ -195,15 +207,20 @@ int ll_gain_norm_add_mix(const float* x, const void* y, int y_dtype, const float
   return LL_OK;
 }
 
-int ll_glu_unit(const void* gu, int gu_stride, int ff, float limit, float alpha, float shift, void* h, int dtype, int rows,
-                ll_stream stream) {
-  LL_CHECK_ARG(gu && h && ff > 0 && gu_stride >= 2 * ff && rows >= 0, "bad glu_unit arguments");
+int ll_glu_unit_rows(const void* gu, int gu_stride, int ff, const float* bias, float limit, float alpha, float shift, void* h,
+                     int h_stride, int dtype, int rows, ll_stream stream) {
+  LL_CHECK_ARG(gu && h && ff > 0 && gu_stride >= 2 * ff && h_stride >= ff && rows >= 0, "bad glu_unit arguments");
   if (rows == 0) return LL_OK;
   cudaStream_t st = (cudaStream_t)stream;
-  if (dtype == LL_F32) return glu_unit_launch<float>(gu, gu_stride, ff, limit, alpha, shift, h, rows, st);
-  if (dtype == LL_BF16) return glu_unit_launch<__nv_bfloat16>(gu, gu_stride, ff, limit, alpha, shift, h, rows, st);
+  if (dtype == LL_F32) return glu_unit_launch<float>(gu, gu_stride, ff, bias, limit, alpha, shift, h, h_stride, rows, st);
+  if (dtype == LL_BF16) return glu_unit_launch<__nv_bfloat16>(gu, gu_stride, ff, bias, limit, alpha, shift, h, h_stride, rows, st);
   set_error("glu_unit: unsupported dtype %d", dtype);
   return LL_ERR_UNSUPPORTED;
+}
+
+int ll_glu_unit(const void* gu, int gu_stride, int ff, float limit, float alpha, float shift, void* h, int dtype, int rows,
+                ll_stream stream) {
+  return ll_glu_unit_rows(gu, gu_stride, ff, nullptr, limit, alpha, shift, h, ff, dtype, rows, stream);
 }
 
 int ll_glu_clamp(const void* gu, int gu_stride, int ff, float limit, float alpha, void* h, int dtype, int rows,
@@ -251,10 +268,11 @@ __global__ void add_norm_pair_kernel(float* __restrict__ x, const TA* __restrict
   }
 }
 
-// x[m][:] += s * a (optional, activation dtype TA), in place, fp32.  Then, if asked for, the layer norm of the same row:
-// out = (x - mean) / sqrt(var + eps) * w + b, var the mean of the squared deviations (formed from the deviations themselves,
-// in a second sweep over the row the block holds).  One block per row; VPT > 0: the row stays in registers, VPT runs of four
-// numbers per thread; VPT = 0: any length, the row in shared memory.
+// x[m][:] += s * (a + a_bias) + step, in place, fp32 (a: optional, activation dtype TA, with an optional fp32 bias row; step: an
+// optional fp32 row).  Then, if asked for, the norm of the same row: the layer norm out = (x - mean) / sqrt(var + eps) * w + b, var
+// the mean of the squared deviations (formed from the deviations themselves, in a second sweep over the row the block holds), or
+// (RMS) out = x / sqrt(mean(x^2) + eps) * w.  One block per row; VPT > 0: the row stays in registers, VPT runs of four numbers per
+// thread; VPT = 0: any length, the row in shared memory.
 template <typename TA> __device__ __forceinline__ float4 ld4(const TA* p);
 template <> __device__ __forceinline__ float4 ld4<float>(const float* p) { return *(const float4*)p; }
 template <> __device__ __forceinline__ float4 ld4<__nv_bfloat16>(const __nv_bfloat16* p) {
@@ -269,45 +287,52 @@ template <> __device__ __forceinline__ void st4<__nv_bfloat16>(__nv_bfloat16* p,
                           (uint32_t)f32_to_bf16_bits(v.z) | ((uint32_t)f32_to_bf16_bits(v.w) << 16));
 }
 
-template <typename TA, int VPT>
-__global__ void add_layer_norm_kernel(float* __restrict__ x, const TA* __restrict__ a, float s, const float* __restrict__ w,
-                                      const float* __restrict__ b, float eps, TA* __restrict__ out, int dim) {
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+
+template <typename TA, int VPT, bool RMS>
+__global__ void add_row_norm_kernel(float* __restrict__ x, const TA* __restrict__ a, float s, const float* __restrict__ a_bias,
+                                    const float* __restrict__ step, const float* __restrict__ w, const float* __restrict__ b, float eps,
+                                    TA* __restrict__ out, int dim) {
   extern __shared__ float ln_row[];
   __shared__ float red[32];
   const size_t base = (size_t)blockIdx.x * dim;
   float sum = 0.f;
   if constexpr (VPT > 0) {
     float4 v[VPT > 0 ? VPT : 1], av[VPT > 0 ? VPT : 1];
+    const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
       const int i = (k * blockDim.x + threadIdx.x) * 4;
-      v[k] = i < dim ? *(const float4*)(x + base + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-      if (a) av[k] = i < dim ? ld4<TA>(a + base + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[k] = i < dim ? *(const float4*)(x + base + i) : zero4;
+      if (a) av[k] = i < dim ? ld4<TA>(a + base + i) : zero4;
     }
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
       const int i = (k * blockDim.x + threadIdx.x) * 4;
       if (a) {
+        if (a_bias && i < dim) av[k] = add4(av[k], *(const float4*)(a_bias + i));
         v[k].x += s * av[k].x, v[k].y += s * av[k].y, v[k].z += s * av[k].z, v[k].w += s * av[k].w;
-        if (i < dim) *(float4*)(x + base + i) = v[k];
       }
-      sum += (v[k].x + v[k].y) + (v[k].z + v[k].w);
+      if (step && i < dim) v[k] = add4(v[k], *(const float4*)(step + i));
+      if ((a || step) && i < dim) *(float4*)(x + base + i) = v[k];
+      if (!RMS) sum += (v[k].x + v[k].y) + (v[k].z + v[k].w);
     }
     if (!out) return;
-    const float mean = block_sum(sum, red) / (float)dim;
+    if constexpr (!RMS) {
+      const float mean = block_sum(sum, red) / (float)dim;
+#pragma unroll
+      for (int k = 0; k < VPT; ++k) v[k].x -= mean, v[k].y -= mean, v[k].z -= mean, v[k].w -= mean;
+    }
     float ss = 0.f;
 #pragma unroll
-    for (int k = 0; k < VPT; ++k) {
-      const int i = (k * blockDim.x + threadIdx.x) * 4;
-      v[k].x -= mean, v[k].y -= mean, v[k].z -= mean, v[k].w -= mean;
-      if (i < dim) ss += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
-    }
+    for (int k = 0; k < VPT; ++k)
+      if ((k * blockDim.x + threadIdx.x) * 4 < dim) ss += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
     const float kn = 1.f / sqrtf(block_sum(ss, red) / (float)dim + eps);
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
       const int i = (k * blockDim.x + threadIdx.x) * 4;
       if (i < dim) {
-        const float4 wv = *(const float4*)(w + i), bv = *(const float4*)(b + i);
+        const float4 wv = *(const float4*)(w + i), bv = RMS ? zero4 : *(const float4*)(b + i);
         st4<TA>(out + base + i, make_float4(v[k].x * kn * wv.x + bv.x, v[k].y * kn * wv.y + bv.y, v[k].z * kn * wv.z + bv.z,
                                             v[k].w * kn * wv.w + bv.w));
       }
@@ -315,30 +340,31 @@ __global__ void add_layer_norm_kernel(float* __restrict__ x, const TA* __restric
   } else {
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {
       float v = x[base + i];
-      if (a) {
-        v += s * dt<TA>::ld(a, base + i);
-        x[base + i] = v;
-      }
+      if (a) v += s * (dt<TA>::ld(a, base + i) + (a_bias ? a_bias[i] : 0.f));
+      if (step) v += step[i];
+      if (a || step) x[base + i] = v;
       ln_row[i] = v;
       sum += v;
     }
     if (!out) return;
-    const float mean = block_sum(sum, red) / (float)dim;
+    const float mean = RMS ? 0.f : block_sum(sum, red) / (float)dim;
     float ss = 0.f;
     for (int i = threadIdx.x; i < dim; i += blockDim.x) {      // (a thread reads back what it wrote itself)
       const float d = ln_row[i] - mean;
       ss += d * d;
     }
     const float kn = 1.f / sqrtf(block_sum(ss, red) / (float)dim + eps);
-    for (int i = threadIdx.x; i < dim; i += blockDim.x) dt<TA>::st(out, base + i, (ln_row[i] - mean) * kn * w[i] + b[i]);
+    for (int i = threadIdx.x; i < dim; i += blockDim.x) dt<TA>::st(out, base + i, (ln_row[i] - mean) * kn * w[i] + (RMS ? 0.f : b[i]));
   }
 }
 
-template <typename TA>
-static int add_layer_norm_launch(float* x, const void* a, float s, const float* w, const float* b, float eps, void* out, int rows, int dim,
-                                 cudaStream_t st) {
-  const bool vec = dim % 4 == 0 && dim <= 8192 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)a | (uintptr_t)out) & 15) == 0;
-#define LL_ALN(VPT, NT, SM) add_layer_norm_kernel<TA, VPT><<<rows, NT, SM, st>>>(x, (const TA*)a, s, w, b, eps, (TA*)out, dim)
+template <typename TA, bool RMS>
+static int add_row_norm_launch(float* x, const void* a, float s, const float* a_bias, const float* step, const float* w, const float* b,
+                               float eps, void* out, int rows, int dim, cudaStream_t st) {
+  const bool vec = dim % 4 == 0 && dim <= 8192 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)a | (uintptr_t)out |
+                                                    (uintptr_t)a_bias | (uintptr_t)step) & 15) == 0;
+#define LL_ALN(VPT, NT, SM) \
+  add_row_norm_kernel<TA, VPT, RMS><<<rows, NT, SM, st>>>(x, (const TA*)a, s, a_bias, step, w, b, eps, (TA*)out, dim)
   if (vec) {
     if (dim <= 2048) LL_ALN(1, (dim / 4 + 31) / 32 * 32, 0);
     else if (dim <= 4096) LL_ALN(2, 512, 0);
@@ -346,18 +372,18 @@ static int add_layer_norm_launch(float* x, const void* a, float s, const float* 
   } else {
     const size_t smem = (size_t)dim * sizeof(float);
     if (smem > 200 * 1024) {
-      set_error("add_layer_norm: rows of %d numbers", dim);
+      set_error("add + norm: rows of %d numbers", dim);
       return LL_ERR_UNSUPPORTED;
     }
     static bool sized = false;
     if (!sized && smem > 48 * 1024) {
-      LL_CUDA(cudaFuncSetAttribute(add_layer_norm_kernel<TA, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+      LL_CUDA(cudaFuncSetAttribute(add_row_norm_kernel<TA, 0, RMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
       sized = true;
     }
     LL_ALN(0, dim >= 512 ? 256 : 128, smem);
   }
 #undef LL_ALN
-  LL_LAUNCH_OK("add_layer_norm_kernel");
+  LL_LAUNCH_OK("add_row_norm_kernel");
   return LL_OK;
 }
 
@@ -372,7 +398,7 @@ static int add_layer_norm_launch(float* x, const void* a, float s, const float* 
 template <typename TA>
 __global__ void gated_group_norm_kernel(const float* __restrict__ y, int y_gs, const float* __restrict__ stab,
                                         const TA* __restrict__ gate, int gate_stride, const float* __restrict__ w, int w_shared,
-                                        float eps, int groups, int gate_first, int gate_sigmoid, TA* __restrict__ out, int C) {
+                                        float eps, int groups, int gate_first, int gate_sigmoid, TA* __restrict__ out, int out_stride, int C) {
   const int m = blockIdx.x;
   const int gs = C / groups;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
@@ -397,7 +423,7 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, int y_gs, c
       const float wv = w[w_shared ? i : g * gs + i];
       const float yv = yr[i] * pre;
       const float v = gate_first ? (yv * sg) * k * wv : yv * k * wv * sg;
-      dt<TA>::st(out, (size_t)m * C + (size_t)g * gs + i, v);
+      dt<TA>::st(out, (size_t)m * out_stride + (size_t)g * gs + i, v);
     }
   }
 }
@@ -407,7 +433,7 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, int y_gs, c
 template <typename TA, int V>
 __global__ void gated_group_norm_wide_kernel(const float* __restrict__ y, const TA* __restrict__ gate, int gate_stride,
                                              const float* __restrict__ w, int w_shared, float eps, int gate_first, int gate_sigmoid,
-                                             TA* __restrict__ out, int gs) {
+                                             TA* __restrict__ out, int out_stride, int gs) {
   extern __shared__ __align__(16) float ggn_row[];
   __shared__ float red[32];
   const size_t m = blockIdx.y;
@@ -415,7 +441,7 @@ __global__ void gated_group_norm_wide_kernel(const float* __restrict__ y, const 
   const float* yr = y + (m * groups + g) * gs;
   const TA* gr = gate + m * gate_stride + (size_t)g * gs;
   const float* wr = w + (w_shared ? 0 : (size_t)g * gs);
-  TA* orow = out + (m * groups + g) * gs;
+  TA* orow = out + m * out_stride + (size_t)g * gs;
   float ss = 0.f;
   auto gated = [&](float v, float z) {
     const float t = v * (gate_sigmoid ? 1.f : z) / (1.f + expf(-z));
@@ -445,8 +471,8 @@ __global__ void gated_group_norm_wide_kernel(const float* __restrict__ y, const 
 
 template <typename TA>
 static int gated_group_norm_wide_launch(const float* y, const void* gate, int gate_stride, const float* w, int w_shared, float eps,
-                                        int groups, int gate_first, int gate_sigmoid, void* out, int rows, int gs, cudaStream_t st) {
-  const bool vec = ((gs | gate_stride) & 3) == 0 && (((uintptr_t)y | (uintptr_t)w | (uintptr_t)out | (uintptr_t)gate) & (4 * sizeof(TA) - 1)) == 0 &&
+                                        int groups, int gate_first, int gate_sigmoid, void* out, int out_stride, int rows, int gs, cudaStream_t st) {
+  const bool vec = ((gs | gate_stride | out_stride) & 3) == 0 && (((uintptr_t)y | (uintptr_t)w | (uintptr_t)out | (uintptr_t)gate) & (4 * sizeof(TA) - 1)) == 0 &&
                    (((uintptr_t)y | (uintptr_t)w) & 15) == 0;
   // few blocks: a thread's share of the row is what the launch takes
   int nt = (long long)rows * groups < 2 * sm_count() ? 1024 : 256;
@@ -454,7 +480,7 @@ static int gated_group_norm_wide_launch(const float* y, const void* gate, int ga
   const size_t smem = (size_t)gs * sizeof(float);
 #define LL_GGN(V)                                                                                                                     \
   gated_group_norm_wide_kernel<TA, V><<<dim3(groups, rows), nt, smem, st>>>(y, (const TA*)gate, gate_stride, w, w_shared, eps, gate_first, \
-                                                                            gate_sigmoid, (TA*)out, gs)
+                                                                            gate_sigmoid, (TA*)out, out_stride, gs)
   if (vec) LL_GGN(4);
   else LL_GGN(1);
 #undef LL_GGN
@@ -713,16 +739,34 @@ int ll_add_layer_norm(float* x, const void* a, float s, const float* w, const fl
   LL_CHECK_ARG(x && rows >= 0 && dim > 0 && (!out || (w && b)), "bad add_layer_norm arguments");
   if (rows == 0) return LL_OK;
   cudaStream_t st = (cudaStream_t)stream;
-  if (act_dtype == LL_F32) return add_layer_norm_launch<float>(x, a, s, w, b, eps, out, rows, dim, st);
-  if (act_dtype == LL_BF16) return add_layer_norm_launch<__nv_bfloat16>(x, a, s, w, b, eps, out, rows, dim, st);
+  if (act_dtype == LL_F32) return add_row_norm_launch<float, false>(x, a, s, nullptr, nullptr, w, b, eps, out, rows, dim, st);
+  if (act_dtype == LL_BF16) return add_row_norm_launch<__nv_bfloat16, false>(x, a, s, nullptr, nullptr, w, b, eps, out, rows, dim, st);
   set_error("add_layer_norm: unsupported dtype %d", act_dtype);
+  return LL_ERR_UNSUPPORTED;
+}
+
+int ll_add_rms_norm(float* x, const void* a, float s, const float* a_bias, const float* step, const float* w, float eps, void* out,
+                    int act_dtype, int rows, int dim, ll_stream stream) {
+  LL_CHECK_ARG(x && rows >= 0 && dim > 0 && (!out || w), "bad add_rms_norm arguments");
+  if (rows == 0) return LL_OK;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (act_dtype == LL_F32) return add_row_norm_launch<float, true>(x, a, s, a_bias, step, w, nullptr, eps, out, rows, dim, st);
+  if (act_dtype == LL_BF16) return add_row_norm_launch<__nv_bfloat16, true>(x, a, s, a_bias, step, w, nullptr, eps, out, rows, dim, st);
+  set_error("add_rms_norm: unsupported dtype %d", act_dtype);
   return LL_ERR_UNSUPPORTED;
 }
 
 int ll_gated_group_norm(const float* y, int y_gs, const float* stab, const void* gate, int gate_stride, const float* w, int w_shared,
                         float eps, int groups, int gate_first, int gate_sigmoid, void* out, int act_dtype, int rows, int C,
                         ll_stream stream) {
-  LL_CHECK_ARG(y && gate && w && out && rows >= 0 && C > 0 && groups > 0 && C % groups == 0 && gate_stride >= C,
+  return ll_gated_group_norm_rows(y, y_gs, stab, gate, gate_stride, w, w_shared, eps, groups, gate_first, gate_sigmoid, out, C, act_dtype,
+                                  rows, C, stream);
+}
+
+int ll_gated_group_norm_rows(const float* y, int y_gs, const float* stab, const void* gate, int gate_stride, const float* w, int w_shared,
+                             float eps, int groups, int gate_first, int gate_sigmoid, void* out, int out_stride, int act_dtype, int rows,
+                             int C, ll_stream stream) {
+  LL_CHECK_ARG(y && gate && w && out && rows >= 0 && C > 0 && groups > 0 && C % groups == 0 && gate_stride >= C && out_stride >= C,
                "bad gated_group_norm arguments");
   if (y_gs == 0) y_gs = C / groups;
   LL_CHECK_ARG(y_gs >= C / groups + (stab ? 1 : 0), "gated_group_norm: a part of y is shorter than the part it norms");
@@ -731,20 +775,21 @@ int ll_gated_group_norm(const float* y, int y_gs, const float* stab, const void*
   const int gs = C / groups;
   if (gs >= 256 && gs <= 12288 && !stab && y_gs == gs && rows <= 65535) {
     if (act_dtype == LL_F32)
-      return gated_group_norm_wide_launch<float>(y, gate, gate_stride, w, w_shared, eps, groups, gate_first, gate_sigmoid, out, rows, gs, st);
+      return gated_group_norm_wide_launch<float>(y, gate, gate_stride, w, w_shared, eps, groups, gate_first, gate_sigmoid, out, out_stride, rows, gs, st);
     if (act_dtype == LL_BF16)
-      return gated_group_norm_wide_launch<__nv_bfloat16>(y, gate, gate_stride, w, w_shared, eps, groups, gate_first, gate_sigmoid, out, rows,
-                                                         gs, st);
+      return gated_group_norm_wide_launch<__nv_bfloat16>(y, gate, gate_stride, w, w_shared, eps, groups, gate_first, gate_sigmoid, out, out_stride,
+                                                         rows, gs, st);
     set_error("gated_group_norm: unsupported dtype %d", act_dtype);
     return LL_ERR_UNSUPPORTED;
   }
   const int threads = groups >= 8 ? 256 : groups >= 4 ? 128 : 32 * groups;
   if (act_dtype == LL_F32)
     gated_group_norm_kernel<float><<<rows, threads, 0, st>>>(y, y_gs, stab, (const float*)gate, gate_stride, w, w_shared, eps, groups,
-                                                            gate_first, gate_sigmoid, (float*)out, C);
+                                                            gate_first, gate_sigmoid, (float*)out, out_stride, C);
   else if (act_dtype == LL_BF16)
     gated_group_norm_kernel<__nv_bfloat16><<<rows, threads, 0, st>>>(y, y_gs, stab, (const __nv_bfloat16*)gate, gate_stride, w, w_shared,
-                                                                    eps, groups, gate_first, gate_sigmoid, (__nv_bfloat16*)out, C);
+                                                                    eps, groups, gate_first, gate_sigmoid, (__nv_bfloat16*)out,
+                                                                    out_stride, C);
   else {
     set_error("gated_group_norm: unsupported dtype %d", act_dtype);
     return LL_ERR_UNSUPPORTED;

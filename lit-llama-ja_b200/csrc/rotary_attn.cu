@@ -268,7 +268,7 @@ __global__ void __launch_bounds__(SA_WARPS * 32) softmax_attn_kernel(
     const T* __restrict__ q, int q_stride, const T* __restrict__ gate, int gate_stride, const T* __restrict__ kc, const T* __restrict__ vc,
     const int32_t* __restrict__ pos_ids, const float* __restrict__ sink, const float* __restrict__ slopes, float scale, float softcap,
     int Tn, int H, int G, int dim, int vdim, int window, int chunk, int ring, int splits, int maps, int pairs, float* __restrict__ part_ml,
-    float* __restrict__ part_acc, T* __restrict__ y) {
+    float* __restrict__ part_acc, T* __restrict__ y, int y_stride) {
   // a warp owns one (query, head, map); with one map per head, h below is the head itself
   const int pair = blockIdx.x * SA_WARPS + (threadIdx.x >> 5);
   if (pair >= pairs) return;
@@ -381,7 +381,7 @@ __global__ void __launch_bounds__(SA_WARPS * 32) softmax_attn_kernel(
       if (c < vdim) {
         float o = acc[r][e] * inv;
         if (gate) o *= 1.f / (1.f + expf(-dt<T>::ld(gate, (size_t)m * gate_stride + (size_t)h * vdim + c)));
-        dt<T>::st(y, (size_t)m * H * vdim + (size_t)h * vdim + c, o);
+        dt<T>::st(y, (size_t)m * y_stride + (size_t)h * vdim + c, o);
       }
     }
 }
@@ -394,7 +394,8 @@ constexpr int SA_MAX_SPLITS = 64;
 template <typename T>
 __global__ void softmax_attn_merge_kernel(const float* __restrict__ part_ml, const float* __restrict__ part_acc,
                                           const T* __restrict__ gate, int gate_stride, const float* __restrict__ sink, int H, int vdim,
-                                          int splits, int maps, float lambda, float post, float eps, int pairs, T* __restrict__ y) {
+                                          int splits, int maps, float lambda, float post, float eps, int pairs, T* __restrict__ y,
+                                          int y_stride) {
   __shared__ float wsp[4][2][SA_MAX_SPLITS];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pair = blockIdx.x * (blockDim.x >> 5) + warp;      // (query, head)
@@ -454,14 +455,14 @@ __global__ void softmax_attn_merge_kernel(const float* __restrict__ part_ml, con
     if (c >= vdim) continue;
     float o = ov[e] * k;
     if (gate) o *= 1.f / (1.f + expf(-dt<T>::ld(gate, (size_t)m * gate_stride + (size_t)h * vdim + c)));
-    dt<T>::st(y, (size_t)m * H * vdim + (size_t)h * vdim + c, o);
+    dt<T>::st(y, (size_t)m * y_stride + (size_t)h * vdim + c, o);
   }
 }
 
 template <typename T, int R, int RV>
 static int sa_launch(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc,
                      const int32_t* pos_ids, const float* sink, const float* slopes, float scale, float softcap, int B, int Tn, int H,
-                     int G, int dim, int vdim, int window, int chunk, int ring, int splits, const DiffMaps& dm, float* scratch, void* y,
+                     int G, int dim, int vdim, int window, int chunk, int ring, int splits, const DiffMaps& dm, float* scratch, void* y, int y_stride,
                      cudaStream_t st) {
   const int pairs = B * Tn * H * dm.maps;
   float* part_ml = scratch;
@@ -469,12 +470,12 @@ static int sa_launch(const void* q, int q_stride, const void* gate, int gate_str
   const dim3 grid((pairs + SA_WARPS - 1) / SA_WARPS, splits);
   softmax_attn_kernel<T, R, RV><<<grid, SA_WARPS * 32, 0, st>>>((const T*)q, q_stride, (const T*)gate, gate_stride, (const T*)kc,
                                                                (const T*)vc, pos_ids, sink, slopes, scale, softcap, Tn, H, G, dim, vdim, window,
-                                                               chunk, ring, splits, dm.maps, pairs, part_ml, part_acc, (T*)y);
+                                                               chunk, ring, splits, dm.maps, pairs, part_ml, part_acc, (T*)y, y_stride);
   LL_LAUNCH_OK("softmax_attn_kernel");
   if (splits > 1 || dm.maps > 1) {
     const int heads = B * Tn * H;
     softmax_attn_merge_kernel<T><<<(heads + 3) / 4, 128, 0, st>>>(part_ml, part_acc, (const T*)gate, gate_stride, sink, H, vdim, splits,
-                                                                 dm.maps, dm.lambda, dm.post, dm.eps, heads, (T*)y);
+                                                                 dm.maps, dm.lambda, dm.post, dm.eps, heads, (T*)y, y_stride);
     LL_LAUNCH_OK("softmax_attn_merge_kernel");
   }
   return LL_OK;
@@ -483,13 +484,13 @@ static int sa_launch(const void* q, int q_stride, const void* gate, int gate_str
 template <typename T>
 static int sa_dispatch(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc,
                        const int32_t* pos_ids, const float* sink, const float* slopes, float scale, float softcap, int B, int Tn, int H,
-                       int G, int dim, int vdim, int window, int chunk, int ring, int splits, const DiffMaps& dm, float* scratch, void* y,
+                       int G, int dim, int vdim, int window, int chunk, int ring, int splits, const DiffMaps& dm, float* scratch, void* y, int y_stride,
                        cudaStream_t st) {
   const int r = dim <= 64 ? 1 : dim <= 128 ? 2 : 4, rv = vdim <= 64 ? 1 : vdim <= 128 ? 2 : 4;
 #define LL_SA(RR, RRV)                                                                                                              \
   if (r == RR && rv == RRV)                                                                                                         \
     return sa_launch<T, RR, RRV>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, slopes, scale, softcap, B, Tn, H, G, dim, vdim, window, \
-                                 chunk, ring, splits, dm, scratch, y, st);
+                                 chunk, ring, splits, dm, scratch, y, y_stride, st);
   LL_SA(1, 1) LL_SA(1, 2) LL_SA(1, 4) LL_SA(2, 1) LL_SA(2, 2) LL_SA(2, 4) LL_SA(4, 1) LL_SA(4, 2) LL_SA(4, 4)
 #undef LL_SA
   return LL_ERR_UNSUPPORTED;
@@ -539,7 +540,7 @@ __global__ void __launch_bounds__(TM_THREADS, MAPS == 1 ? 3 : 2) softmax_attn_mm
     const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ gate, int gate_stride,
     const __nv_bfloat16* __restrict__ kc, const __nv_bfloat16* __restrict__ vc, const int32_t* __restrict__ pos_ids,
     const float* __restrict__ sink, const float* __restrict__ slopes, float scale, float softcap, int Tn, int H, int G, int dim, int vdim,
-    int window, int chunk, int ring, float lambda, float post, float eps, __nv_bfloat16* __restrict__ y) {
+    int window, int chunk, int ring, float lambda, float post, float eps, __nv_bfloat16* __restrict__ y, int y_stride) {
   constexpr int LD = DK + 8, CH = DK / 8, LV = DV + 8, CV = DV / 8, STAGE = TM_K * (LD + LV);      // a stage: 64 key rows, then 64 value rows
   extern __shared__ __align__(16) unsigned char tm_smem[];
   __nv_bfloat16* const stages = (__nv_bfloat16*)tm_smem;
@@ -739,7 +740,7 @@ __global__ void __launch_bounds__(TM_THREADS, MAPS == 1 ? 3 : 2) softmax_attn_mm
           v0 *= 1.f / (1.f + expf(-__bfloat162float(gg.x)));
           v1 *= 1.f / (1.f + expf(-__bfloat162float(gg.y)));
         }
-        *(__nv_bfloat162*)(y + m * H * vdim + (size_t)h * vdim + c) = __floats2bfloat162_rn(v0, v1);
+        *(__nv_bfloat162*)(y + m * y_stride + (size_t)h * vdim + c) = __floats2bfloat162_rn(v0, v1);
       }
     }
   }
@@ -750,7 +751,7 @@ template <int DK, int DV, int MAPS, bool BIAS = false>
 static int tm_launch(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, const int32_t* pos_ids,
                      const float* sink, const float* slopes, float scale, float softcap, int B, int Tn, int H, int G, int dim, int vdim,
                      int window, int chunk,
-                     int ring, const DiffMaps& dm, void* y, cudaStream_t st) {
+                     int ring, const DiffMaps& dm, void* y, int y_stride, cudaStream_t st) {
   const dim3 grid((Tn + TM_Q - 1) / TM_Q, H, B);
   constexpr int smem = 2 * TM_K * (DK + 8 + DV + 8) * (int)sizeof(__nv_bfloat16);
   static bool sized = false;
@@ -760,7 +761,7 @@ static int tm_launch(const void* q, int q_stride, const void* gate, int gate_str
   }
   softmax_attn_mma_kernel<DK, DV, MAPS, BIAS><<<grid, TM_THREADS, smem, st>>>(
       (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)gate, gate_stride, (const __nv_bfloat16*)kc, (const __nv_bfloat16*)vc,
-      pos_ids, sink, slopes, scale, softcap, Tn, H, G, dim, vdim, window, chunk, ring, dm.lambda, dm.post, dm.eps, (__nv_bfloat16*)y);
+      pos_ids, sink, slopes, scale, softcap, Tn, H, G, dim, vdim, window, chunk, ring, dm.lambda, dm.post, dm.eps, (__nv_bfloat16*)y, y_stride);
   LL_LAUNCH_OK("softmax_attn_mma_kernel");
   return LL_OK;
 }
@@ -863,11 +864,11 @@ size_t ll_softmax_attn_scratch_bytes(int M, int H, int vdim, int splits) {
   return (size_t)M * H * splits * (2 + (size_t)vdim) * sizeof(float);
 }
 
-int ll_softmax_attn_biased(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, int dtype,
-                           const int32_t* pos_ids, const float* sink, const float* slopes, float scale, float softcap, int B, int T, int H,
-                           int G, int dim, int vdim, int window, int chunk, int ring, int splits, int form, int maps, float diff_lambda,
-                           float diff_post, float eps, float* scratch, void* y, ll_stream stream) {
-  LL_CHECK_ARG(q && kc && vc && pos_ids && y, "softmax_attn: null pointer");
+int ll_softmax_attn_rows(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, int dtype,
+                         const int32_t* pos_ids, const float* sink, const float* slopes, float scale, float softcap, int B, int T, int H,
+                         int G, int dim, int vdim, int window, int chunk, int ring, int splits, int form, int maps, float diff_lambda,
+                         float diff_post, float eps, float* scratch, void* y, int y_stride, ll_stream stream) {
+  LL_CHECK_ARG(q && kc && vc && pos_ids && y && y_stride >= H * vdim, "softmax_attn: null pointer or short output rows");
   LL_CHECK_ARG(B >= 0 && T >= 0 && H > 0 && G > 0 && H % G == 0 && dim > 0 && vdim > 0 && ring > 0 && window >= 0 && chunk >= 0 &&
                    splits >= 1 && splits <= SA_MAX_SPLITS && (maps == 1 || maps == 2),
                "bad softmax_attn arguments");
@@ -878,12 +879,13 @@ int ll_softmax_attn_biased(const void* q, int q_stride, const void* gate, int ga
   if (B == 0 || T == 0) return LL_OK;
   cudaStream_t st = (cudaStream_t)stream;
   const DiffMaps dm{maps, diff_lambda, diff_post, eps};
-  if (form == 0 && !(slopes && maps > 1) && tm_supported(dtype, T, dim, vdim, q_stride, gate ? gate_stride : 0, splits)) {
+  if (form == 0 && !(slopes && maps > 1) && tm_supported(dtype, T, dim, vdim, q_stride, gate ? gate_stride : 0, splits) &&
+      y_stride % 2 == 0) {
     const int d = dim > vdim ? dim : vdim;
     if (maps == 1) {           // one map: key and value rows padded alike
 #define LL_TM_B(DD, BB)                                                                                                               \
   tm_launch<DD, DD, 1, BB>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, slopes, scale, softcap, B, T, H, G, dim, vdim, window, \
-                           chunk, ring, dm, y, st)
+                           chunk, ring, dm, y, y_stride, st)
 #define LL_TM(DD) \
   if (d <= DD) return slopes ? LL_TM_B(DD, true) : LL_TM_B(DD, false);
       LL_TM(32) LL_TM(64) LL_TM(96) LL_TM(128)
@@ -893,7 +895,7 @@ int ll_softmax_attn_biased(const void* q, int q_stride, const void* gate, int ga
 #define LL_TM2(KK, VV)                                                                                                              \
   if (dim <= KK && vdim <= VV)                                                                                                      \
     return tm_launch<KK, VV, 2>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, slopes, scale, softcap, B, T, H, G, dim, vdim, window, \
-                                chunk, ring, dm, y, st);
+                                chunk, ring, dm, y, y_stride, st);
 #define LL_TM2_ROW(KK) LL_TM2(KK, 32) LL_TM2(KK, 64) LL_TM2(KK, 96) LL_TM2(KK, 128)
     LL_TM2_ROW(32) LL_TM2_ROW(64) LL_TM2_ROW(96) LL_TM2_ROW(128)
 #undef LL_TM2_ROW
@@ -902,12 +904,20 @@ int ll_softmax_attn_biased(const void* q, int q_stride, const void* gate, int ga
   LL_CHECK_ARG(scratch || (splits == 1 && maps == 1), "softmax_attn: split key ranges and several maps meet in scratch memory");
   if (dtype == LL_F32)
     return sa_dispatch<float>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, slopes, scale, softcap, B, T, H, G, dim, vdim, window, chunk,
-                              ring, splits, dm, scratch, y, st);
+                              ring, splits, dm, scratch, y, y_stride, st);
   if (dtype == LL_BF16)
     return sa_dispatch<__nv_bfloat16>(q, q_stride, gate, gate_stride, kc, vc, pos_ids, sink, slopes, scale, softcap, B, T, H, G, dim, vdim, window,
-                                      chunk, ring, splits, dm, scratch, y, st);
+                                      chunk, ring, splits, dm, scratch, y, y_stride, st);
   set_error("softmax_attn: unsupported dtype %d", dtype);
   return LL_ERR_UNSUPPORTED;
+}
+
+int ll_softmax_attn_biased(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, int dtype,
+                           const int32_t* pos_ids, const float* sink, const float* slopes, float scale, float softcap, int B, int T, int H,
+                           int G, int dim, int vdim, int window, int chunk, int ring, int splits, int form, int maps, float diff_lambda,
+                           float diff_post, float eps, float* scratch, void* y, ll_stream stream) {
+  return ll_softmax_attn_rows(q, q_stride, gate, gate_stride, kc, vc, dtype, pos_ids, sink, slopes, scale, softcap, B, T, H, G, dim, vdim,
+                              window, chunk, ring, splits, form, maps, diff_lambda, diff_post, eps, scratch, y, H * vdim, stream);
 }
 
 int ll_softmax_attn_maps(const void* q, int q_stride, const void* gate, int gate_stride, const void* kc, const void* vc, int dtype,

@@ -111,6 +111,9 @@ EXPORTS = {
     "ll_gain_norm_add_mix": ([vp, vp, i32, vp, C.c_float, vp, vp, sz_t, vp, i32, vp, vp, i32, i32, i32, vp], C.c_int),
     "ll_glu_clamp": ([vp, i32, i32, C.c_float, C.c_float, vp, i32, i32, vp], C.c_int),
     "ll_glu_unit": ([vp, i32, i32, C.c_float, C.c_float, C.c_float, vp, i32, i32, vp], C.c_int),
+    "ll_glu_unit_rows": ([vp, i32, i32, vp, C.c_float, C.c_float, C.c_float, vp, i32, i32, i32, vp], C.c_int),
+    "ll_latent_attn_terms": ([vp, i64, i64, vp, i32, i32, i32, i32, vp, vp, vp, vp, i64, i64, i32, i32, i32, i32, i32, i32, i32, i32,
+                              i32, C.c_float, i32, i32, vp, vp], C.c_int),
     "ll_latent_kv_append": ([vp, i32, i32, i32, vp, C.c_float, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp], C.c_int),
     "ll_latent_attn": ([vp, i64, i64, vp, i32, i32, i32, i32, vp, vp, vp, vp, i64, i64, i32, i32, i32, i32, i32, i32, i32, i32,
                         i32, C.c_float, i32, vp, vp], C.c_int),
@@ -126,6 +129,8 @@ EXPORTS = {
     "ll_add_norm_pair": ([vp, vp, C.c_float, vp, C.c_float, vp, C.c_float, vp, vp, C.c_float, vp, i32, vp, i32, i32, i32, vp], C.c_int),
     "ll_add_layer_norm": ([vp, vp, C.c_float, vp, vp, C.c_float, vp, i32, i32, i32, vp], C.c_int),
     "ll_gated_group_norm": ([vp, i32, vp, vp, i32, vp, i32, C.c_float, i32, i32, i32, vp, i32, i32, i32, vp], C.c_int),
+    "ll_add_rms_norm": ([vp, vp, C.c_float, vp, vp, vp, C.c_float, vp, i32, i32, i32, vp], C.c_int),
+    "ll_gated_group_norm_rows": ([vp, i32, vp, vp, i32, vp, i32, C.c_float, i32, i32, i32, vp, i32, i32, i32, i32, vp], C.c_int),
     "ll_gelu": ([vp, i32, i32, sz_t, vp], C.c_int),
     "ll_relu_squared": ([vp, i32, sz_t, vp], C.c_int),
     "ll_short_conv": ([vp, i32, i32, i32, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp], C.c_int),
@@ -151,6 +156,14 @@ EXPORTS = {
                            i32, i32, i32, i32, i32, i32, i32, vp], C.c_int),
     "ll_softmax_attn_biased": ([vp, i32, vp, i32, vp, vp, i32, vp, vp, vp, C.c_float, C.c_float, i32, i32, i32, i32, i32, i32, i32, i32,
                                 i32, i32, i32, i32, C.c_float, C.c_float, C.c_float, vp, vp, vp], C.c_int),
+    "ll_softmax_attn_rows": ([vp, i32, vp, i32, vp, vp, i32, vp, vp, vp, C.c_float, C.c_float, i32, i32, i32, i32, i32, i32, i32, i32,
+                              i32, i32, i32, i32, C.c_float, C.c_float, C.c_float, vp, vp, i32, vp], C.c_int),
+    "ll_delta_scan": ([vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, vp, vp, C.c_float, C.c_float, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
+                      C.c_int),
+    "ll_delta_chunked_supported": ([i32, i32, i32, i32, i32, i32, i32], C.c_int),
+    "ll_delta_chunked_scratch_bytes": ([i32, i32, i32, i32, i32], sz_t),
+    "ll_delta_chunked": ([vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, vp, vp, C.c_float, C.c_float, vp, vp, vp, i32, i32, i32, i32, i32, i32,
+                          vp, vp], C.c_int),
     "ll_hyper_mix_norm": ([vp, i64, i64, vp, vp, vp, C.c_float, vp, vp, vp, vp, C.c_float, vp, i32, vp, i32, i32, i32, i32, vp], C.c_int),
     "ll_row_norm": ([vp, i32, vp, C.c_float, vp, i32, i32, i32, i32, vp], C.c_int),
     "ll_sigmoid_gate_mul": ([vp, i32, vp, i32, vp, i32, i32, i32, i32, vp], C.c_int),
@@ -164,7 +177,7 @@ EXPORTS = {
 }
 _fn = {name: _proto(name, a, r) for name, (a, r) in EXPORTS.items()}
 
-ABI_VERSION = 16
+ABI_VERSION = 17
 if _fn["ll_abi_version"]() != ABI_VERSION:
     raise ImportError("libllb200.so ABI version mismatch; rebuild with lit-llama-ja_b200/build.py")
 

@@ -19,6 +19,7 @@ Variations, all parameters of the spec:
 * ``rot_layout``: "interleaved" pairs dimension 2i with 2i+1; "half" pairs i with i + rot_dims/2.  The kernels turn
   interleaved pairs; a "half" checkpoint has the rows of its rotated query and key parts reordered once at load time (the
   same reordering on both sides of the dot product leaves the scores as they are).
+* ``exact_weights``: in bf16 the softmax weights enter the weighted sum as two bf16 terms (16 bits) instead of one.
 * ``rotary``: a ``rotary.RotarySpec`` whose ``table()`` (rescaled frequencies, magnitude) replaces the plain table.
 """
 from __future__ import annotations
@@ -51,6 +52,7 @@ class LatentAttentionSpec:
     q_rank: Optional[int] = None     # queries through a normed latent of this size; None: q = W_q h
     gate: str = "head"               # "head" | "element" | "none"
     rot_layout: str = "interleaved"  # "interleaved" | "half"
+    exact_weights: bool = False      # softmax weights as two bf16 terms in the tensor-core form
     rotary: Optional[RotarySpec] = None   # rescaled frequencies and magnitude; None: base^(-2i/rot_dims)
 
     def __post_init__(self):
@@ -103,7 +105,7 @@ def build_rope_table(n_pos: int, rot_dims: int, base: float, device) -> torch.Te
 
 
 class LatentAttention(nn.Module):
-    def __init__(self, spec: LatentAttentionSpec, dtype: torch.dtype, device) -> None:
+    def __init__(self, spec: LatentAttentionSpec, dtype: torch.dtype, device, project: bool = True) -> None:
         super().__init__()
         s = self.spec = spec
         self.owns_cache = s.kv_from is None
@@ -115,39 +117,57 @@ class LatentAttention(nn.Module):
         self.n_in = n_in
         n_in = (n_in + 7) // 8 * 8          # rows of zeros up to a multiple of 8: the library's fast GEMMs want aligned outputs
         kw = dict(dtype=dtype, device=device)
-        self.w_in = nn.Parameter(torch.empty((n_in, s.width), **kw), requires_grad=False)          # [W_q | W_dq; W_g; W_dkv]
+        # [W_q | W_dq; W_g; W_dkv]; project False: the layer keeps the input and output projections, stacked with others
+        self.w_in = nn.Parameter(torch.empty((n_in, s.width), **kw), requires_grad=False) if project else None
         self.q_norm = nn.Parameter(torch.ones(s.q_rank, dtype=torch.float32, device=device), requires_grad=False) \
             if s.q_rank is not None else None
         self.w_uq = nn.Parameter(torch.empty((self.q_cols, s.q_rank), **kw), requires_grad=False) if s.q_rank is not None else None
         self.w_uk = nn.Parameter(torch.empty((s.heads, s.nope_dim, s.kv_rank), **kw), requires_grad=False)
         self.w_uv_t = nn.Parameter(torch.empty((s.heads, s.kv_rank, s.v_dim), **kw), requires_grad=False)
-        self.w_o = nn.Parameter(torch.empty((s.width, s.heads * s.v_dim), **kw), requires_grad=False)
+        self.w_o = nn.Parameter(torch.empty((s.width, s.heads * s.v_dim), **kw), requires_grad=False) if project else None
         self.kv_norm = nn.Parameter(torch.ones(s.kv_rank, dtype=torch.float32, device=device), requires_grad=False) \
             if self.owns_cache else None
 
-    def load(self, get) -> None:
-        """``get(suffix)`` returns the tensor '<layer>.mix.<suffix>' ([out, in] for the Linears)."""
+    @property
+    def out_cols(self) -> int:
+        """What ``attend`` puts out per token."""
+        return self.spec.heads * self.spec.v_dim
+
+    def state_shapes(self, B: int):
+        return []
+
+    def cache_shapes(self, B: int, ring: int):
+        return [(B, ring, self.spec.row)] if self.owns_cache else []
+
+    def _q_rows(self, w: torch.Tensor) -> torch.Tensor:
+        """The rotated part of every head's query rows in the stored order."""
         s = self.spec
-        order = s.rot_order()
+        w = w.reshape(s.heads, s.q_head, -1)
+        return torch.cat([w[:, : s.nope_dim], w[:, s.nope_dim:][:, s.rot_order()]], dim=1).reshape(self.q_cols, -1)
 
-        def q_rows(w):                      # the rotated part of every head's query rows in the stored order
-            w = w.reshape(s.heads, s.q_head, -1)
-            return torch.cat([w[:, : s.nope_dim], w[:, s.nope_dim:][:, order]], dim=1).reshape(self.q_cols, -1)
-
-        parts = [get("dq")] if s.q_rank is not None else [q_rows(get("q"))]
+    def in_rows(self, get) -> torch.Tensor:
+        """The rows of the input projection."""
+        s = self.spec
+        parts = [get("dq")] if s.q_rank is not None else [self._q_rows(get("q"))]
         if s.gate != "none":
             parts.append(get("g"))
         if self.owns_cache:
             dkv = get("dkv")
-            parts.append(torch.cat([dkv[: s.kv_rank], dkv[s.kv_rank:][order]], dim=0))
-        self.w_in.zero_()
-        self.w_in[: self.n_in].copy_(torch.cat([p.to(self.w_in.dtype) for p in parts], dim=0))
+            parts.append(torch.cat([dkv[: s.kv_rank], dkv[s.kv_rank:][s.rot_order()]], dim=0))
+        return torch.cat(parts, dim=0)
+
+    def load(self, get) -> None:
+        """``get(suffix)`` returns the tensor '<layer>.mix.<suffix>' ([out, in] for the Linears)."""
+        s = self.spec
+        if self.w_in is not None:
+            self.w_in.zero_()
+            self.w_in[: self.n_in].copy_(self.in_rows(get))
+            self.w_o.copy_(get("o"))
         if s.q_rank is not None:
             self.q_norm.copy_(get("dq.norm").float())
-            self.w_uq.copy_(q_rows(get("uq")))
+            self.w_uq.copy_(self._q_rows(get("uq")))
         self.w_uk.copy_(get("uk").reshape(s.heads, s.nope_dim, s.kv_rank))
         self.w_uv_t.copy_(get("uv").reshape(s.heads, s.v_dim, s.kv_rank).transpose(1, 2))
-        self.w_o.copy_(get("o"))
         if self.owns_cache:
             self.kv_norm.copy_(get("dkv.norm").float())
 
@@ -155,18 +175,24 @@ class LatentAttention(nn.Module):
                 splits: int = 1) -> torch.Tensor:
         """x_act ``[B*T, width]`` -> ``[B*T, width]``; ``cache`` ``[B, S, row]`` is this layer's or its source's (already
         appended to by the source in this step)."""
+        return F.linear(self.attend(F.linear(x_act, self.w_in), B, T, pos_ids, rope, cache, splits), self.w_o)
+
+    def attend(self, proj: torch.Tensor, B: int, T: int, pos_ids: torch.Tensor, rope: torch.Tensor, cache: torch.Tensor,
+               splits: int = 1, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``proj``: the input projection's output (this mixer's columns first).  Returns the gated heads
+        ``[B*T, heads * v_dim]`` before the output projection, in ``out`` (a column slice) when given."""
         s = self.spec
         M = B * T
-        dt = N.dtype_code(x_act.dtype)
+        dt = N.dtype_code(proj.dtype)
         st = N.stream()
-        proj = F.linear(x_act, self.w_in)                                     # [M, n_in]
+        dev = proj.device
         S = cache.shape[1]
         if self.owns_cache:
-            N.call("ll_latent_kv_append", N.ptr(proj), dt, proj.shape[1], self.kv_col0, N.ptr(self.kv_norm), float(s.eps),
+            N.call("ll_latent_kv_append", N.ptr(proj), dt, proj.stride(0), self.kv_col0, N.ptr(self.kv_norm), float(s.eps),
                    N.ptr(rope), N.ptr(pos_ids), N.ptr(cache), B, T, s.kv_rank, s.rot_dim, s.rot_dims, S, st)
         if s.q_rank is not None:
-            cq = torch.empty((M, s.q_rank), dtype=x_act.dtype, device=x_act.device)
-            N.call("ll_row_norm", N.ptr(proj), proj.shape[1], N.ptr(self.q_norm), float(s.eps), N.ptr(cq), s.q_rank, dt, M, s.q_rank, st)
+            cq = torch.empty((M, s.q_rank), dtype=proj.dtype, device=dev)
+            N.call("ll_row_norm", N.ptr(proj), proj.stride(0), N.ptr(self.q_norm), float(s.eps), N.ptr(cq), s.q_rank, dt, M, s.q_rank, st)
             q = F.linear(cq, self.w_uq)                                       # [M, heads * q_head]
         else:
             q = proj
@@ -176,16 +202,20 @@ class LatentAttention(nn.Module):
         scratch = None
         if splits > 1:
             scratch = torch.empty(N.call_ret("ll_latent_attn_scratch_bytes", M, s.heads, s.kv_rank, splits) // 4,
-                                  dtype=torch.float32, device=x_act.device)
+                                  dtype=torch.float32, device=dev)
         head_gate = self.gate_col0 if (s.gate == "head" and s.q_rank is None) else -1
-        N.call("ll_latent_attn", N.ptr(q_lat), M * s.kv_rank, s.kv_rank, N.ptr(q), q.shape[1], s.nope_dim, s.q_head,
+        N.call("ll_latent_attn_terms", N.ptr(q_lat), M * s.kv_rank, s.kv_rank, N.ptr(q), q.stride(0), s.nope_dim, s.q_head,
                head_gate, N.ptr(rope), N.ptr(pos_ids), N.ptr(cache), N.ptr(o_lat), M * s.kv_rank, s.kv_rank, dt, B, T,
                s.heads, s.kv_rank, s.rot_dim, s.rot_dims, S, s.window if s.window is not None else 0, float(s.scale), splits,
-               N.ptr(scratch), st)
-        o = torch.bmm(o_lat, self.w_uv_t).transpose(0, 1).reshape(M, s.heads * s.v_dim)     # [M, heads * v_dim]
+               2 if s.exact_weights else 1, N.ptr(scratch), st)
+        if out is not None:                    # the heads' products land where they belong in the rows
+            o = out
+            torch.bmm(o_lat, self.w_uv_t, out=o.view(M, s.heads, s.v_dim).transpose(0, 1))
+        else:
+            o = torch.bmm(o_lat, self.w_uv_t).transpose(0, 1).reshape(M, s.heads * s.v_dim)     # [M, heads * v_dim]
         if s.gate == "element":
-            N.call("ll_sigmoid_gate_mul", N.ptr(o), o.shape[1], N.ptr_at(proj, self.gate_col0), proj.shape[1], N.ptr(o), o.shape[1], dt,
+            N.call("ll_sigmoid_gate_mul", N.ptr(o), o.stride(0), N.ptr_at(proj, self.gate_col0), proj.stride(0), N.ptr(o), o.stride(0), dt,
                    M, s.heads * s.v_dim, st)
         elif s.gate == "head" and s.q_rank is not None:
             raise NotImplementedError("a gate per head beside latent queries")
-        return F.linear(o, self.w_o)
+        return o

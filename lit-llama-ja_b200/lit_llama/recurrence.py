@@ -17,6 +17,12 @@
       q, k, v = silu(W_q h), silu(W_k h), silu(W_v h);  S_t = decay_h S_(t-1) + k_t v_t^T;  o_t = S_t^T q_t
       out = W_o ( rmsnorm(all heads together) * w * sigmoid(W_g h) )
 
+* ``GatedDeltaMixer`` - gated delta rule (csrc/delta_rule.cu, csrc/delta_chunk.cu): what the faded memory returns for a key is
+  compared with the value, and the difference is written under that key:
+      q, k, v = silu(shortconv(W h));  q, k <- unit vectors per head;  q <- q * dim^(-1/2)
+      g = exp(-exp(A_log) softplus(W_a h + dt_bias));  beta = sigmoid(W_b h)
+      S <- g S;  S <- S + k (beta (v - S^T k))^T;  o = S^T q;   out = W_o ( headnorm(o) * w * silu(W_g h) )
+
 Prompts in bfloat16 whose decay is one number per head and token (or a constant per head) run in chunks of 64 tokens on tensor
 cores (csrc/decay_chunk.cu); single tokens, short portions, fp32 and decays per channel walk token by token
 (csrc/decay_scan.cu).  Decays, step sizes, the state, the read-out and the norms are fp32; the projections, the short convolution's output and
@@ -86,14 +92,34 @@ def decay_scan_constant(proj, q_col, k_col, v_col, decay, silu, qscale, state, p
     return y
 
 
-def gated_group_norm(y, gate, gate_col, weight, shared, eps, groups, gate_first, out_dtype, sigmoid=False, part=None, stab=None):
+def delta_scan(q, q_col, k, k_col, v, v_col, gates, a_col, b_col, dt_bias, a_log, unit_eps, qscale, state, pos_ids, B, T, H, qk_heads, n, p):
+    """fp32 ``[B*T, H*p]``: the read-out of the gated delta rule (see csrc/delta_rule.cu) over column slices of matrices in the
+    activation dtype (``gates``: the projections that give the decay, at ``a_col``, and the write strength, at ``b_col``);
+    ``state`` is advanced in place."""
+    y = torch.empty((B * T, H * p), dtype=torch.float32, device=v.device)
+    args = (N.ptr_at(q, q_col), q.stride(0), N.ptr_at(k, k_col), k.stride(0), N.ptr_at(v, v_col), v.stride(0), N.ptr_at(gates, a_col),
+            N.ptr_at(gates, b_col), gates.stride(0), N.dtype_code(v.dtype), N.ptr(dt_bias), N.ptr(a_log), float(unit_eps), float(qscale),
+            N.ptr(state), N.ptr(pos_ids), N.ptr(y), B, T, H, qk_heads, n, p)
+    slices = ((q, q_col), (k, k_col), (v, v_col))
+    if (USE_CHUNKS and N.has("ll_delta_chunked")
+            and bool(N.call_ret("ll_delta_chunked_supported", N.dtype_code(v.dtype), T, n, p, q.stride(0), k.stride(0), v.stride(0)))
+            and all((x.data_ptr() + c * x.element_size()) % 16 == 0 for x, c in slices)):
+        scratch = torch.empty(N.call_ret("ll_delta_chunked_scratch_bytes", B, T, H, n, p) // 4, dtype=torch.float32, device=v.device)
+        N.call("ll_delta_chunked", *args, N.ptr(scratch), N.stream())
+    else:
+        N.call("ll_delta_scan", *args, N.stream())
+    return y
+
+
+def gated_group_norm(y, gate, gate_col, weight, shared, eps, groups, gate_first, out_dtype, sigmoid=False, part=None, stab=None, out=None):
     """``y`` fp32 ``[rows, groups * part]`` (``part`` None: the parts are what is normed, nothing between them); see
-    csrc/residual_ops.cu for ``stab``."""
+    csrc/residual_ops.cu for ``stab``; ``out``: a column slice to write to."""
     C = y.shape[1] if part is None else groups * part
-    out = torch.empty((y.shape[0], C), dtype=out_dtype, device=y.device)
-    N.call("ll_gated_group_norm", N.ptr(y), y.shape[1] // groups, N.ptr(stab), N.ptr_at(gate, gate_col), gate.stride(0), N.ptr(weight),
-           1 if shared else 0, float(eps), groups, 1 if gate_first else 0, 1 if sigmoid else 0, N.ptr(out), N.dtype_code(out_dtype),
-           y.shape[0], C, N.stream())
+    if out is None:
+        out = torch.empty((y.shape[0], C), dtype=out_dtype, device=y.device)
+    N.call("ll_gated_group_norm_rows", N.ptr(y), y.shape[1] // groups, N.ptr(stab), N.ptr_at(gate, gate_col), gate.stride(0), N.ptr(weight),
+           1 if shared else 0, float(eps), groups, 1 if gate_first else 0, 1 if sigmoid else 0, N.ptr(out), out.stride(0),
+           N.dtype_code(out_dtype), y.shape[0], C, N.stream())
     return out
 
 
@@ -330,3 +356,85 @@ class ConstantDecayAttention(nn.Module):
                                 s.vdim)
         out = gated_group_norm(y, proj, c["g"], self.norm, False, s.eps, 1, False, proj.dtype, sigmoid=True)
         return F.linear(out, self.w_o)
+
+
+@dataclass
+class GatedDeltaSpec:
+    width: int
+    heads: int              # value heads
+    kv_heads: int           # query / key heads, each shared by heads / kv_heads consecutive value heads
+    dim: int                # query / key channels per head
+    vdim: int
+    taps: int
+    eps: float
+    unit_eps: float = 1e-6
+
+    def __post_init__(self):
+        if self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} heads over {self.kv_heads} query/key heads")
+
+
+class GatedDeltaMixer(nn.Module):
+    """``project`` False: the layer keeps the input and output projections itself (stacked with others)."""
+
+    def __init__(self, spec: GatedDeltaSpec, dtype: torch.dtype, device, project: bool = True) -> None:
+        super().__init__()
+        s = self.spec = spec
+        kw = dict(dtype=dtype, device=device)
+        f32 = dict(dtype=torch.float32, device=device)
+        gd, hv = s.kv_heads * s.dim, s.heads * s.vdim
+        self.cols = dict(q=0, k=gd, v=2 * gd, g=pad8(2 * gd + hv))
+        self.cols["a"] = self.cols["g"] + hv
+        self.cols["b"] = self.cols["a"] + s.heads
+        self.n_in = self.cols["b"] + s.heads
+        self.w_in = nn.Parameter(torch.zeros((pad8(self.n_in), s.width), **kw), requires_grad=False) if project else None
+        self.conv = ShortConv(2 * gd + hv, s.taps, False, device)              # q, k and v side by side
+        self.dt_bias = nn.Parameter(torch.zeros(s.heads, **f32), requires_grad=False)
+        self.a_log = nn.Parameter(torch.zeros(s.heads, **f32), requires_grad=False)
+        self.norm = nn.Parameter(torch.ones(s.vdim, **f32), requires_grad=False)
+        self.w_o = nn.Parameter(torch.zeros((s.width, hv), **kw), requires_grad=False) if project else None
+
+    @property
+    def out_cols(self) -> int:
+        return self.spec.heads * self.spec.vdim
+
+    def state_shapes(self, B: int) -> List[Tuple[int, ...]]:
+        """fp32: the convolution's inputs, the memory."""
+        s = self.spec
+        return [self.conv.state_shape(B), (B, s.heads, s.dim, s.vdim)]
+
+    def cache_shapes(self, B: int, ring: int) -> List[Tuple[int, ...]]:
+        return []
+
+    def in_rows(self, get) -> torch.Tensor:
+        q = get("q")
+        rows = torch.zeros((self.n_in, q.shape[1]), dtype=q.dtype, device=q.device)
+        for name, at in self.cols.items():
+            w = get(name)
+            rows[at: at + w.shape[0]] = w
+        return rows
+
+    def load(self, get) -> None:
+        """``get(suffix)`` returns the tensor '<layer>.mix.<suffix>'."""
+        if self.w_in is not None:
+            self.w_in.zero_()
+            self.w_in[: self.n_in].copy_(self.in_rows(get))
+            self.w_o.copy_(get("o"))
+        self.conv.load(torch.cat([get(n + ".conv").float() for n in "qkv"], dim=0))
+        self.dt_bias.copy_(get("dt_bias").float())
+        self.a_log.copy_(get("A_log").float())
+        self.norm.copy_(get("norm").float())
+
+    def forward(self, u: torch.Tensor, B: int, T: int, pos_ids: torch.Tensor, states) -> torch.Tensor:
+        return F.linear(self.mix(F.linear(u, self.w_in), B, T, pos_ids, states), self.w_o)
+
+    def mix(self, proj: torch.Tensor, B: int, T: int, pos_ids: torch.Tensor, states, out=None) -> torch.Tensor:
+        """``proj``: the input projection's output (this mixer's columns first).  Returns ``[B*T, heads * vdim]`` before the
+        output projection, in ``out`` (a column slice) when given."""
+        s = self.spec
+        c = self.cols
+        conv_state, memory = states
+        qkv = self.conv(proj, 0, conv_state, pos_ids, B, T, proj.dtype, silu=True)
+        y = delta_scan(qkv, c["q"], qkv, c["k"], qkv, c["v"], proj, c["a"], c["b"], self.dt_bias, self.a_log, s.unit_eps, s.dim ** -0.5, memory,
+                       pos_ids, B, T, s.heads, s.kv_heads, s.dim, s.vdim)
+        return gated_group_norm(y, proj, c["g"], self.norm, True, s.eps, s.heads, False, proj.dtype, out=out)

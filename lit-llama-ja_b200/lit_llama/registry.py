@@ -47,6 +47,10 @@ def _builtin() -> None:
         from .livasun import ARCHITECTURE, Livasun
 
         register_architecture(ARCHITECTURE, Livasun.from_dir)
+    if "Zekonex" not in _FROM_DIR:
+        from .zekonex import ARCHITECTURE, Zekonex
+
+        register_architecture(ARCHITECTURE, Zekonex.from_dir)
 
 
 def load_model_dir(path, dtype: torch.dtype = torch.bfloat16, device="cuda"):

@@ -11,6 +11,7 @@ from __future__ import annotations
 import contextlib
 import gc
 import os
+from dataclasses import astuple
 from typing import Dict, List, Optional, Tuple
 
 import torch
@@ -18,6 +19,7 @@ import torch.nn as nn
 
 from . import _native as N
 from .cache import TensorPool, max_portion, ring_length
+from .rotary import RotarySpec
 
 
 @contextlib.contextmanager
@@ -145,9 +147,9 @@ class PortionedDecoder(nn.Module):
 
 
 class RingStateDecoder(PortionedDecoder):
-    """A model whose per-sequence memory is fp32 recurrent state (``states``: every layer's tensors in order) and key / value
-    rings in the activation dtype (``kv_caches``: (keys, values) of every ring in order), each as long as the furthest look-back
-    among its readers and a pass of ``prefill_portion`` tokens ask for.  All of it comes from the package's ``TensorPool`` with
+    """A model whose per-sequence memory is fp32 recurrent state (``states``: every layer's tensors in order) and rings in the
+    activation dtype (``kv_caches``: the tensors of every ring in order, keys and values or latent rows), each as long as the
+    furthest look-back among its readers and a pass of ``prefill_portion`` tokens ask for.  All of it comes from the package's ``TensorPool`` with
     stable addresses and is written in place; nothing is cleared between requests: the kernels start a sequence from nothing
     when its first position is 0.  A model sets ``config``, ``dtype``, ``device`` and says what its memory looks like."""
 
@@ -158,14 +160,20 @@ class RingStateDecoder(PortionedDecoder):
         self.kv_caches: List[torch.Tensor] = []
         self._rings: Tuple[int, ...] = ()
         self._batch = 0
+        self._rope: Dict[tuple, torch.Tensor] = {}     # (cos, sin) tables for kernels that look the turn up
+        self._rope_len = 0
 
     # ------------------------------------------------------------------ hooks
+    def _rotary_specs(self) -> List[RotarySpec]:
+        """The rotations whose tables (``rope_table``) the layers look up."""
+        return []
+
     def _ring_reaches(self) -> List[Optional[int]]:
         """Per ring: no reader's query at position i sees a key before ``i - reach + 1`` (None: unbounded)."""
         raise NotImplementedError
 
     def _ring_shapes(self, n: int, B: int, ring: int) -> List[Tuple[int, ...]]:
-        """(keys, values) of ring ``n`` with ``ring`` slots."""
+        """The tensors of ring ``n`` with ``ring`` slots."""
         raise NotImplementedError
 
     def _state_shapes(self, B: int) -> List[Tuple[int, ...]]:
@@ -181,7 +189,21 @@ class RingStateDecoder(PortionedDecoder):
         portion = min(self.prefill_portion, max_seq_length)
         return tuple(max(1, ring_length(max_seq_length, r, portion)) for r in self._ring_reaches())
 
+    def rope_table(self, spec: RotarySpec) -> torch.Tensor:
+        return self._rope[astuple(spec)]
+
+    def _ensure_rope(self, n_pos: int) -> None:
+        specs = self._rotary_specs()
+        if not specs or n_pos <= self._rope_len:
+            return
+        n = max(n_pos, 2 * self._rope_len, 1024)
+        for spec in specs:
+            self._rope[astuple(spec)] = spec.table(n, self.device)
+        self._rope_len = n
+        self._drop_graphs()
+
     def _begin(self, B: int, max_seq_length: int, keep: bool) -> None:
+        self._ensure_rope(max_seq_length)
         rings = self._ring_plan(max_seq_length)
         if (self.states or self.kv_caches) and self._batch == B and self._rings == rings:
             return
@@ -245,6 +267,13 @@ def add_layer_norm(x, branch, scale, w, b, eps, out, act_dtype) -> None:
     """``x += scale * branch`` in place (fp32; ``branch`` None: nothing is added); then, with ``out`` given, ``out`` = the layer
     norm of ``x`` with weight ``w`` and bias ``b``."""
     N.call("ll_add_layer_norm", N.ptr(x), N.ptr(branch), float(scale), N.ptr(w), N.ptr(b), float(eps), N.ptr(out),
+           N.dtype_code(act_dtype), x.shape[0], x.shape[1], N.stream())
+
+
+def add_rms_norm(x, branch, scale, bias, step, w, eps, out, act_dtype) -> None:
+    """``x += scale * (branch + bias) + step`` in place (fp32; ``bias`` an fp32 row beside the branch, ``step`` an fp32 row that joins
+    every row of the stream; each may be None); then, with ``out`` given, ``out = rmsnorm(x) * w``."""
+    N.call("ll_add_rms_norm", N.ptr(x), N.ptr(branch), float(scale), N.ptr(bias), N.ptr(step), N.ptr(w), float(eps), N.ptr(out),
            N.dtype_code(act_dtype), x.shape[0], x.shape[1], N.stream())
 
 

@@ -128,7 +128,7 @@ __global__ void __launch_bounds__(DC_THREADS, 3) delta_prepare_kernel(const Delt
       ss += x0 * x0 + x1 * x1;
     }
     ss = warp_sum(ss);
-    if (lane == 0) rk[t] = 1.f / sqrtf(ss + A.unit_eps);
+    if (lane == 0) rk[t] = t < len ? 1.f / sqrtf(ss + A.unit_eps) : 0.f;
   }
   __syncthreads();
   if (tid < DC_L) {
@@ -174,6 +174,11 @@ __global__ void __launch_bounds__(DC_THREADS, 3) delta_prepare_kernel(const Delt
       for (int k = 0; k < i; ++k) v = fmaf(-L[(r + i) * DX_LD + r + k], x[k], v);
       x[i] = v;
       X[(r + i) * DX_LD + r + cc] = v;
+    }
+  } else {            // meanwhile the zeros right of them that the merge of the halves reads
+    for (int i = tid - DC_L; i < 512; i += DC_THREADS - DC_L) {
+      const int r = (i >> 8) * 32 + ((i >> 4) & 15), cc = (i >> 8) * 32 + 16 + (i & 15);
+      X[r * DX_LD + cc] = 0.f;
     }
   }
   __syncthreads();

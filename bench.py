@@ -49,7 +49,7 @@ def parse():
     ap.add_argument("--steps", type=int, default=3)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
-    ap.add_argument("--family", default=None, choices=[None, "lepalorn", "bededra", "tebodra", "bumulix", "livasun"],
+    ap.add_argument("--family", default=None, choices=[None, "lepalorn", "bededra", "tebodra", "bumulix", "livasun", "zekonex"],
                     help="instead of the headline workload: prefill / decode throughput and kernel rooflines of this model family "
                          "beside its closest relative at equal size (lepalorn beside LLaMA, bededra beside lepalorn, tebodra beside bededra, "
                          "bumulix beside tebodra, livasun beside bededra; 1 GPU; one JSON line of its own)")

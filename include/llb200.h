@@ -575,6 +575,8 @@ LL_API int ll_delta_chunked(const void* q, int q_stride, const void* k, int k_st
                             const void* raw_b, int gate_stride, int dtype, const float* dt_bias, const float* a_log, float unit_eps,
                             float qs, float* state, const int32_t* pos_ids, float* y, int B, int T, int H, int qk_heads, int n, int p,
                             float* scratch, ll_stream stream);
+/* 0, or 1 when a bounded wait inside these kernels ran out since the library was loaded (synchronises the device). */
+LL_API int ll_delta_chunk_error(void);
 /* Exponential gates with a running stabiliser, per (b, h): li = cap(raw_i + bias_i[h]), lf = logsigmoid(cap(raw_f + bias_f[h])),
  * cap(z) = c tanh(z / c) (c <= 0: none); mx_t = max(lf_t + mx_(t-1), li_t) with mx carried in mstate fp32 [B][H] (0 when
  * pos_ids[0] == 0); keep = exp(lf + mx_(t-1) - mx_t), take = exp(li - mx_t), stab = mx_t   (fp32 [B*T][H] each). */

@@ -1,7 +1,7 @@
 """Throughput of a model family beside its closest relative at equal size: prefill tokens/s, batch-1 decode tokens/s, and
 the hot kernels of each timed alone against the measured roofline.  ``bench.py --family lepalorn``: Lepalorn beside LLaMA;
 ``bench.py --family bededra``: Bededra beside Lepalorn; ``bench.py --family tebodra``: Tebodra beside Bededra; ``--family bumulix``: Bumulix beside Tebodra; ``--family livasun``: Livasun
-beside Bededra.  Random weights, layer shapes of real
+beside Bededra; ``--family zekonex``: Zekonex beside Bumulix, its recurrence beside Livasun's.  Random weights, layer shapes of real
 models, a few layers each (every layer costs the same).  Timing: CUDA events, warm-up, an L2 flush (a 256 MB write)
 between timed iterations."""
 from __future__ import annotations
@@ -901,12 +901,184 @@ def run_livasun(args):
     return 0
 
 
+# Zekonex at the widths of SIZES, four layers each: softmax attention over the whole past, delta rule, latent attention, delta rule.
+# Attention heads as Livasun's, latent attention as Bumulix's (without latent queries), the delta rule with as many 128 x 128 heads as
+# Livasun's linear attention, two of them on one query / key head; a clamped unit on every layer whose three matrices are the size of
+# Bumulix's two (ff = 8/3 width).
+ZEKONEX_SIZES = {
+    "w1024": dict(width=1024, layers=4, heads=8, kv=2, dim=64, d_heads=8, d_dim=128, l_heads=8, nope=64, rot=32, v=64, kv_rank=256, ff=2688),
+    "w2048": dict(width=2048, layers=4, heads=16, kv=4, dim=128, d_heads=16, d_dim=128, l_heads=16, nope=128, rot=64, v=128, kv_rank=512, ff=5440),
+    "w4096": dict(width=4096, layers=4, heads=32, kv=8, dim=128, d_heads=32, d_dim=128, l_heads=32, nope=128, rot=64, v=128, kv_rank=512, ff=10880),
+}
+
+
+def zekonex_model(s, device, dtype=torch.bfloat16):
+    from lit_llama.zekonex import Zekonex, ZekonexConfig
+
+    ff = {"kind": "dense", "ff": s["ff"], "limit": 7.0}
+    att = {"type": "attention", "mlp": ff, "mixer": {"heads": s["heads"], "kv_heads": s["kv"], "dim": s["dim"], "vdim": s["dim"],
+                                                     "rot": {"base": 10000.0, "dims": s["dim"] // 2}, "scale": s["dim"] ** -0.5}}
+    dlt = {"type": "delta", "mlp": ff, "mixer": {"heads": s["d_heads"], "kv_heads": s["d_heads"] // 2, "dim": s["d_dim"], "vdim": s["d_dim"],
+                                                 "conv": 4}}
+    lat = {"type": "latent_attention", "mlp": ff, "mixer": {
+        "heads": s["l_heads"], "dim": s["nope"], "rot_dim": s["rot"], "vdim": s["v"], "kv_rank": s["kv_rank"],
+        "rot": {"base": 10000.0, "dims": s["rot"]}, "scale": (s["nope"] + s["rot"]) ** -0.5}}
+    cfg = {"vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.5, "embedding": {"scale": 1.0},
+           "layers": [att, dlt, lat, dlt][: s["layers"]]}
+    m = Zekonex(ZekonexConfig.from_dict(cfg), dtype=dtype, device=device)
+    g = torch.Generator(device=device).manual_seed(0)
+    fixed = {"dt_bias": -2.0, "a_log": 0.0}
+    for n, p in m.named_parameters():
+        leaf = n.rsplit(".", 1)[-1]
+        if p.dim() >= 2 and "conv" not in n:
+            p.copy_((torch.randn(p.shape, generator=g, device=device) / math.sqrt(p.shape[-1])).to(p.dtype))
+        elif p.dim() >= 2:
+            p.copy_(0.5 * torch.randn(p.shape, generator=g, device=device))
+        elif leaf in fixed:
+            p.fill_(fixed[leaf])
+    return m.eval()
+
+
+def zekonex_kernel_table(s, model, device, timer, prompt_len):
+    """The kernels of one layer of each kind alone.  Roofline time = max(flops / tensor peak, bytes / copy bandwidth), flops and
+    bytes counted for the mechanism (one sweep over the visible keys; per token one read, one update and one read-out of the
+    memory)."""
+    from torch.nn import functional as F
+
+    from lit_llama import _native as N
+    from lit_llama.recurrence import delta_scan
+    from lit_llama.stepping import add_rms_norm
+
+    hbm, tflops, which = peaks()
+    bf = torch.bfloat16
+    rows = []
+
+    def add(name, t, flops, nbytes):
+        roof = max(flops / tflops, nbytes / hbm)
+        rows.append(dict(kernel=name, us=round(t * 1e6, 1), roofline_us=round(roof * 1e6, 2), fraction=round(roof / t, 4)))
+
+    E, ff = s["width"], s["ff"]
+    first = {}
+    for r in model.runs:
+        first.setdefault(r.block.kind, r)
+    sms = torch.cuda.get_device_properties(device).multi_processor_count
+    for T, tag in ((prompt_len, "prefill"), (1, "decode")):
+        pos0 = 0 if T > 1 else prompt_len
+        pos_ids = torch.arange(pos0, pos0 + T, dtype=torch.int32, device=device)
+        model.reset_cache()
+        model._begin(1, prompt_len + 64, True)
+        for t in model.kv_caches:
+            t.normal_()
+        for t in model.states:
+            t.zero_()
+        x = torch.randn((T, E), device=device, dtype=bf)
+        keys = sum(p + 1 for p in range(pos0, pos0 + T))
+        # softmax attention
+        run = first["attention"]
+        att, sp = run.block.mix, run.block.mix.spec
+        H, G, D = sp.heads, sp.kv_heads, sp.dim
+        proj = F.linear(x, run.block.w_in)
+        out = torch.empty((T, run.block.n_out), device=device, dtype=bf)
+        caches = model.kv_caches[run.cache_at:run.cache_at + 2]
+        splits = 1 if T > 1 else max(1, min(64, (2 * sms) // max(1, (H + 3) // 4), (caches[0].shape[1] + 31) // 32))
+        add(f"attention {tag} (rotation + append + attention with sink)",
+            timer(lambda: att.attend(proj, 1, T, pos_ids, caches, None, splits, out=out[:, : att.out_cols]), graph=True),
+            2.0 * keys * H * 2 * D, 2.0 * ((pos0 + T) * G * 2 * D + T * (2 * H * D + 2 * G * D)))
+        # delta rule
+        run = first["delta"]
+        dm, ds = run.block.mix, run.block.mix.spec
+        c = dm.cols
+        pd = F.linear(x, run.block.w_in)
+        conv_state, memory = model.states[run.state_at:run.state_at + 2]
+        qkv = dm.conv(pd, 0, conv_state, pos_ids, 1, T, bf, silu=True)
+        nst = ds.heads * ds.dim * ds.vdim
+        y = torch.randn((T, ds.heads * ds.vdim), device=device)
+        add(f"delta rule {tag}",
+            timer(lambda: delta_scan(qkv, c["q"], qkv, c["k"], qkv, c["v"], pd, c["a"], c["b"], dm.dt_bias, dm.a_log, ds.unit_eps,
+                                     ds.dim ** -0.5, memory, pos_ids, 1, T, ds.heads, ds.kv_heads, ds.dim, ds.vdim), graph=True),
+            6.0 * T * nst, 2.0 * T * (2 * ds.kv_heads * ds.dim + ds.heads * ds.vdim + 2 * ds.heads) + 4.0 * T * ds.heads * ds.vdim + 8.0 * nst)
+        add(f"short_conv {tag} (q, k, v with silu)", timer(lambda: dm.conv(pd, 0, conv_state, pos_ids, 1, T, bf, silu=True), graph=True), 0.0,
+            T * dm.conv.channels * 4.0)
+        gated_norm_row(f"gated norm {tag} (delta rule, per head)", y, pd, c["g"], dm.norm, True, ds.heads, False, False, timer, add)
+        # latent attention
+        run = first["latent_attention"]
+        lat, ls = run.block.mix, run.block.mix.spec
+        cache, rope = model.kv_caches[run.cache_at], model.rope_table(ls.rotary)
+        pl = F.linear(x, run.block.w_in)
+        q_lat = torch.randn((ls.heads, T, ls.kv_rank), dtype=bf, device=device)
+        o_lat = torch.empty_like(q_lat)
+        lsplits = 1 if T > 1 else max(1, min(16, (2 * sms) // max(1, (ls.heads + 31) // 32), (cache.shape[1] + 63) // 64))
+        scratch = torch.empty(N.call_ret("ll_latent_attn_scratch_bytes", T, ls.heads, ls.kv_rank, lsplits) // 4 + 4, device=device)
+        dt = N.dtype_code(bf)
+
+        def latent_kernels():
+            st = N.stream()
+            N.call("ll_latent_kv_append", N.ptr(pl), dt, pl.stride(0), lat.kv_col0, N.ptr(lat.kv_norm), 1e-5, N.ptr(rope), N.ptr(pos_ids),
+                   N.ptr(cache), 1, T, ls.kv_rank, ls.rot_dim, ls.rot_dims, cache.shape[1], st)
+            N.call("ll_latent_attn_terms", N.ptr(q_lat), T * ls.kv_rank, ls.kv_rank, N.ptr(pl), pl.stride(0), ls.nope_dim, ls.q_head, -1,
+                   N.ptr(rope), N.ptr(pos_ids), N.ptr(cache), N.ptr(o_lat), T * ls.kv_rank, ls.kv_rank, dt, 1, T, ls.heads, ls.kv_rank,
+                   ls.rot_dim, ls.rot_dims, cache.shape[1], 0, float(ls.scale), lsplits, 2, N.ptr(scratch), st)
+
+        add(f"latent attention {tag} (latent norm + append + attention in latent space, two-term weights)", timer(latent_kernels, graph=True),
+            2.0 * keys * ls.heads * (2 * ls.kv_rank + ls.rot_dim),
+            2.0 * ((pos0 + T) * ls.row + T * ls.heads * (2 * ls.kv_rank + ls.rot_dim)))
+        # stream and feed-forward
+        blk = run.block
+        xs, a0, h = torch.randn((T, E), device=device), torch.randn((T, E), device=device, dtype=bf), torch.empty((T, E), device=device, dtype=bf)
+        add(f"add + rms norm {tag} (with the bias)",
+            timer(lambda: add_rms_norm(xs, a0, 0.5, blk.mlp.bias_down, None, blk.norm1, 1e-5, h, bf), graph=True), 0.0, T * E * (4 + 4 + 2 + 2))
+        rows_out = torch.empty((T, blk.n_out), device=device, dtype=bf)
+        add(f"clamped unit {tag} (biases, strided rows)",
+            timer(lambda: blk.mlp(pl[:, blk.ff_in:], rows_out[:, blk.ff_out: blk.ff_out + ff]), graph=True), 0.0, T * ff * 6)
+    return rows, which
+
+
+def run_zekonex(args):
+    import sys
+
+    sys.path.insert(0, str(ROOT))
+    from __graft_entry__ import build
+
+    build()
+    device = torch.device("cuda", 0)
+    torch.cuda.set_device(device)
+    timer = Timer(device)
+    prompt_len = 2048
+    out = {"family": "zekonex", "beside": "bumulix", "dtype": "bf16", "data": "synthetic (random weights)", "prompt_len": prompt_len,
+           "batch": 1, "l2": "256 MB written between timed iterations", "sizes": {}}
+    for name in [n for n in ZEKONEX_SIZES if not getattr(args, "size", None) or n == args.size]:
+        s = ZEKONEX_SIZES[name]
+        with torch.no_grad():
+            m = zekonex_model(s, device)
+            pre, dec = end_to_end(m, timer, prompt_len, device, prompt_len + 64)
+            rows, which = zekonex_kernel_table(s, m, device, timer, prompt_len)
+            del m
+            torch.cuda.empty_cache()
+            bs = dict(BUMULIX_SIZES[name], layers=s["layers"])
+            bum = bumulix_model(bs, device)
+            bpre, bdec = end_to_end(bum, timer, prompt_len, device, prompt_len + 64)
+            brows, _ = bumulix_kernel_table(bs, bum, device, timer, prompt_len)
+            del bum
+            torch.cuda.empty_cache()
+            ls = dict(LIVASUN_SIZES[name], layers=s["layers"])
+            liv = livasun_model(ls, device)
+            lrows, _ = livasun_kernel_table(ls, liv, device, timer, prompt_len)
+            del liv
+            torch.cuda.empty_cache()
+        out["sizes"][name] = {"config": s, "zekonex": {"prefill_tokens_per_s": round(pre), "decode_tokens_per_s": round(dec, 1)},
+                              "bumulix_same_width": {"prefill_tokens_per_s": round(bpre), "decode_tokens_per_s": round(bdec, 1)},
+                              "kernels": rows, "bumulix_kernels": brows, "livasun_kernels": lrows, "roofline": f"of {which}"}
+    print(json.dumps(out))
+    return 0
+
+
 def run(args):
     import sys
 
+    if args.family == "zekonex":
+        return run_zekonex(args)
     if args.family == "livasun":
         return run_livasun(args)
-
     if args.family == "bededra":
         return run_bededra(args)
     if args.family == "tebodra":

@@ -21,6 +21,12 @@ __device__ __forceinline__ void dc_ldmatrix_trans(uint32_t (&r)[4], const void* 
 __device__ __forceinline__ void dc_ldmatrix_trans2(uint32_t& r0, uint32_t& r1, const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(smem_u32(p)));
 }
+// D(16x8,f32) += A(16x16,bf16,row) * B(16x8,bf16,col); a function of registers alone, which the compiler may move between loads
+__device__ __forceinline__ void dc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
 // x as bf16 terms: the first of (a, b) packed, the rest left in a and b
 __device__ __forceinline__ uint32_t dc_term(float& a, float& b) {
   const uint32_t u = pack_bf16(a, b);

@@ -428,6 +428,62 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ y, int y_gs, c
   }
 }
 
+// The same for short parts in multiples of four numbers without a normaliser: a warp per (row, part), VPT float4 a lane, the part in
+// registers between the two sweeps.
+template <typename TA, int VPT>
+__global__ void __launch_bounds__(256) gated_group_norm4_kernel(const float* __restrict__ y, int y_gs, const TA* __restrict__ gate,
+                                                                int gate_stride, const float* __restrict__ w, int w_shared, float eps,
+                                                                int groups, int gate_first, int gate_sigmoid, TA* __restrict__ out,
+                                                                int out_stride, int gs, int parts) {
+  const int part = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (part >= parts) return;
+  const int m = part / groups, g = part - m * groups;
+  const float* yr = y + (size_t)part * y_gs;
+  const TA* gr = gate + (size_t)m * gate_stride + (size_t)g * gs;
+  const float* wr = w + (w_shared ? 0 : (size_t)g * gs);
+  float4 v[VPT], z[VPT];
+  float ss = 0.f;
+  auto gated = [&](float t) { return (gate_sigmoid ? 1.f : t) / (1.f + expf(-t)); };
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = (k * 32 + lane) * 4;
+    v[k] = i < gs ? *(const float4*)(yr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    z[k] = i < gs ? ld4<TA>(gr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    z[k] = make_float4(gated(z[k].x), gated(z[k].y), gated(z[k].z), gated(z[k].w));
+    const float4 t = make_float4(v[k].x * z[k].x, v[k].y * z[k].y, v[k].z * z[k].z, v[k].w * z[k].w);
+    const float4 n = gate_first ? t : v[k];
+    ss += (n.x * n.x + n.y * n.y) + (n.z * n.z + n.w * n.w);
+    v[k] = t;
+  }
+  const float kn = 1.f / sqrtf(warp_sum(ss) / (float)gs + eps);
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = (k * 32 + lane) * 4;
+    if (i >= gs) continue;
+    const float4 wv = *(const float4*)(wr + i);
+    st4<TA>(out + (size_t)m * out_stride + (size_t)g * gs + i, make_float4(v[k].x * kn * wv.x, v[k].y * kn * wv.y, v[k].z * kn * wv.z,
+                                                                          v[k].w * kn * wv.w));
+  }
+}
+
+template <typename TA>
+static int gated_group_norm4_launch(const float* y, int y_gs, const void* gate, int gate_stride, const float* w, int w_shared, float eps,
+                                    int groups, int gate_first, int gate_sigmoid, void* out, int out_stride, int rows, int gs,
+                                    cudaStream_t st) {
+  const int parts = rows * groups;
+#define LL_GGN4(VPT)                                                                                                                  \
+  gated_group_norm4_kernel<TA, VPT><<<(parts + 7) / 8, 256, 0, st>>>(y, y_gs, (const TA*)gate, gate_stride, w, w_shared, eps, groups, \
+                                                                     gate_first, gate_sigmoid, (TA*)out, out_stride, gs, parts)
+  if (gs <= 128) LL_GGN4(1);
+  else LL_GGN4(2);
+#undef LL_GGN4
+  LL_LAUNCH_OK("gated_group_norm4_kernel");
+  return LL_OK;
+}
+
 // The same for long parts (a whole row of heads normed together): a block per (row, part), the gated numbers of the first sweep
 // kept in shared memory.  V numbers at a time per thread (4: rows and parts on 4-number boundaries).
 template <typename TA, int V>
@@ -781,6 +837,16 @@ int ll_gated_group_norm_rows(const float* y, int y_gs, const float* stab, const 
                                                          rows, gs, st);
     set_error("gated_group_norm: unsupported dtype %d", act_dtype);
     return LL_ERR_UNSUPPORTED;
+  }
+  const uintptr_t at16 = (uintptr_t)y | (uintptr_t)w, at_act = (uintptr_t)gate | (uintptr_t)out;
+  if (!stab && gs <= 256 && ((gs | y_gs | gate_stride | out_stride) & 3) == 0 && (at16 & 15) == 0 &&
+      (at_act & (act_dtype == LL_F32 ? 15 : 7)) == 0 && (long long)rows * groups < (1ll << 31)) {
+    if (act_dtype == LL_F32)
+      return gated_group_norm4_launch<float>(y, y_gs, gate, gate_stride, w, w_shared, eps, groups, gate_first, gate_sigmoid, out, out_stride,
+                                             rows, gs, st);
+    if (act_dtype == LL_BF16)
+      return gated_group_norm4_launch<__nv_bfloat16>(y, y_gs, gate, gate_stride, w, w_shared, eps, groups, gate_first, gate_sigmoid, out,
+                                                     out_stride, rows, gs, st);
   }
   const int threads = groups >= 8 ? 256 : groups >= 4 ? 128 : 32 * groups;
   if (act_dtype == LL_F32)

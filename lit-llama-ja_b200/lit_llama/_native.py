@@ -164,6 +164,7 @@ EXPORTS = {
     "ll_delta_chunked_scratch_bytes": ([i32, i32, i32, i32, i32], sz_t),
     "ll_delta_chunked": ([vp, i32, vp, i32, vp, i32, vp, vp, i32, i32, vp, vp, C.c_float, C.c_float, vp, vp, vp, i32, i32, i32, i32, i32, i32,
                           vp, vp], C.c_int),
+    "ll_delta_chunk_error": ([], C.c_int),
     "ll_hyper_mix_norm": ([vp, i64, i64, vp, vp, vp, C.c_float, vp, vp, vp, vp, C.c_float, vp, i32, vp, i32, i32, i32, i32, vp], C.c_int),
     "ll_row_norm": ([vp, i32, vp, C.c_float, vp, i32, i32, i32, i32, vp], C.c_int),
     "ll_sigmoid_gate_mul": ([vp, i32, vp, i32, vp, i32, i32, i32, i32, vp], C.c_int),

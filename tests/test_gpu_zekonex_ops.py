@@ -221,7 +221,7 @@ def test_delta_rule_walk_in_portions(H, G, n, p, repeat, dtype):
         close(state[0], S, 2e-5)
 
 
-@pytest.mark.parametrize("H,G,n,p", [(2, 1, 8, 8), (4, 2, 16, 24), (3, 3, 40, 64), (4, 2, 64, 72), (2, 2, 128, 136), (6, 1, 104, 16), (40, 20, 24, 96)])
+@pytest.mark.parametrize("H,G,n,p", [(2, 1, 8, 8), (4, 2, 16, 24), (3, 3, 40, 64), (4, 2, 64, 72), (2, 2, 128, 136), (6, 1, 104, 16), (16, 8, 64, 136), (40, 20, 24, 96)])
 @pytest.mark.parametrize("repeat", [False, True])
 def test_delta_rule_in_chunks(H, G, n, p, repeat):
     """Chunk edges, last chunks that are not full, steps that begin inside a sequence, a decay of zero and one of one in the middle of a
@@ -242,6 +242,7 @@ def test_delta_rule_in_chunks(H, G, n, p, repeat):
         state = torch.full((1, H, n, p), float("nan"), device="cuda")
         close(run_delta(case, H, G, n, p, portions, bf, qs, state), want, 5e-5)      # (16 bits where fp32 factors meet each other)
         close(state[0], S, 5e-5)
+    assert N.call_ret("ll_delta_chunk_error") == 0              # no wait for a copy ran out
 
 
 def test_chunks_and_walk_agree_on_identical_keys(monkeypatch):

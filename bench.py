@@ -52,7 +52,7 @@ def parse():
     ap.add_argument("--family", default=None, choices=[None, "lepalorn", "bededra", "tebodra", "bumulix", "livasun", "zekonex"],
                     help="instead of the headline workload: prefill / decode throughput and kernel rooflines of this model family "
                          "beside its closest relative at equal size (lepalorn beside LLaMA, bededra beside lepalorn, tebodra beside bededra, "
-                         "bumulix beside tebodra, livasun beside bededra; 1 GPU; one JSON line of its own)")
+                         "bumulix beside tebodra, livasun beside bededra, zekonex beside bumulix; 1 GPU; one JSON line of its own)")
     ap.add_argument("--size", default=None, help="with --family: one of the family's sizes (default: all)")
     return ap.parse_args()
 
